@@ -442,12 +442,18 @@ typedef enum {
     B200_MIXER_SSD = 7,          /* state-space mixer with a scalar decay per head and token (Mamba-2): short causal convolution on x, B
                                     and C, a softplus step size per head, fp32 matrix state [state, vdim] per head, a skip term, the
                                     result gated by silu(z) and RMS-normed in equal groups                                           */
-    B200_MIXER_LINEAR = 8        /* linear attention with ONE constant decay per head: silu on q, k and v, fp32 matrix state per head,
+    B200_MIXER_LINEAR = 8,       /* linear attention with ONE constant decay per head: silu on q, k and v, fp32 matrix state per head,
                                     RMS norm over the concatenated heads, sigmoid output gate                                        */
+    B200_MIXER_MINGRU = 9        /* gated recurrence whose gates read the current token only (minGRU), an fp32 VECTOR state:
+                                    s <- (1 - z) s + z c,  z = sigmoid(z-in),  c = u + 1/2 where u >= 0, sigmoid(u) elsewhere;
+                                    result s * silu(gate)                                                                             */
 } b200_mixer_kind_t;
 typedef enum { B200_ATTN_SOFTMAX = 0, B200_ATTN_SIGMOID = 1 } b200_attn_weight_t;
 typedef enum { B200_MLP_NONE = 0, B200_MLP_MOE = 1, B200_MLP_DENSE = 2 } b200_mlp_kind_t;
-typedef enum { B200_ACT_RELU2 = 0, B200_ACT_SILU = 1, B200_ACT_GELU_TANH = 2, B200_ACT_RELU = 3 } b200_act_t;
+typedef enum { B200_ACT_RELU2 = 0, B200_ACT_SILU = 1, B200_ACT_GELU_TANH = 2, B200_ACT_RELU = 3,
+    B200_ACT_POLYNORM = 4, /* DENSE, not gated: a n(z) + b n(z^2) + c n(z^3) + e, powers element by element, n(v) = v / rms(v) over the row   */
+    B200_ACT_CLAMP_GLU = 5 /* gated only: g = min(gate, limit), u = clamp(up, -limit, limit): g * sigmoid(slope * g) * (u + 1)                */
+} b200_act_t;
 typedef enum {
     B200_NORM_RMS_POST = 0,      /* x += rmsnorm(sublayer(x)) * g                                                                     */
     B200_NORM_DYT_PRE_POST = 1,  /* x += ls * dyt_b(sublayer(dyt_a(x))), dyt(v) = tanh(alpha v) * w + b: no mean, no variance         */
@@ -455,13 +461,17 @@ typedef enum {
                                     sublayers read it.  Their input projections are one matrix (w_in: mixer rows, side mixer rows,
                                     then the feed-forward's gate rows and up rows) and so are their output projections (w_out
                                     [width, mixer columns | side mixer columns | expert_ff]); w_up / w_down stay NULL                 */
-    B200_NORM_LN_PRE = 3         /* pre-norm with two layer norms (pre1 / pre2, packed [w | b]): x += mixer(ln1(x)); x += ff(ln2(x)).
+    B200_NORM_LN_PRE = 3,        /* pre-norm with two layer norms (pre1 / pre2, packed [w | b]): x += mixer(ln1(x)); x += ff(ln2(x)).
                                     With residual streams (config streams >= 1 and hc1 / hc2 set) a sublayer reads u = sum_s in[s] x_s
                                     and all streams are rewritten at once: x_t <- sum_s mix[s][t] x_s + out[t] * sublayer(ln(u)); the
                                     model's result is the sum of the streams.  w_in holds the mixer's rows, then the side mixer's;
                                     every mixer has an output projection of its own (w_out; side->w_out); with branch_norm set, the
                                     mixer sublayer's result is mix_scale * rmsnorm(mixer) * branch_norm + side_scale * rmsnorm(side) *
                                     side->branch_norm.  Feed-forward: DENSE, gated (w_up [2*expert_ff, width]: gate rows, then up rows) */
+    B200_NORM_RMS_SUM = 4        /* the norm takes the SUM: x <- rmsnorm(residual_scale * x + mixer(x')) * norm1, then the same with the
+                                    feed-forward and norm2.  A sublayer reads x' = x + conv(x), a causal convolution over time on every
+                                    channel (in_taps, in_conv1 / in_conv2; in_taps == 0: x' = x); its last in_taps - 1 inputs are
+                                    part of a sequence's state                                                                        */
 } b200_norm_kind_t;
 typedef enum {
     B200_ROUTE_SIGMOID = 0,      /* scores = sigmoid(logits), the chosen scores are the weights, applied to the expert's INPUT        */
@@ -485,6 +495,9 @@ typedef struct {
                            0: every layer runs once                                                                                  */
     float logit_scale;  /* logits <- logits * logit_scale (before the soft cap); 0 reads as 1                                         */
     int streams;        /* LN_PRE layers: residual streams (1 .. 8); 0 reads as 1                                                     */
+    float pos_base;     /* RMS_SUM layers: > 0: a sinusoidal position vector joins the embedding: channels 2i, 2i + 1 receive sin, cos of
+                           p * pos_base^(-2i / width); 0: none                                                                        */
+    float residual_scale; /* RMS_SUM layers: see B200_NORM_RMS_SUM                                                                    */
 } b200_hybrid_config_t;
 
 typedef struct b200_hybrid_layer_s {
@@ -507,7 +520,7 @@ typedef struct b200_hybrid_layer_s {
     const void *w_decay; const float *decay_bias; /* GLA: [heads*dim, decay_rank], [heads*dim]                                        */
     const float *out_norm;        /* GLA: [vdim], shared by the heads                                                                 */
     const float *norm1, *norm2;   /* RMS_POST: [width]                                                                                */
-    const void *w_router;         /* MOE: SIGMOID: [experts + 1, width]: router rows, then the shared expert's gate row (zeros if none);
+    const void *w_router;         /* MOE: SIGMOID: [experts, width], with a shared expert [experts + 1, width]: its gate row comes last;
                                      SOFTMAX: [experts + identity, width]                                                            */
     const void *w_up, *w_down;    /* MOE: [experts, expert_ff, width] ([experts, 2*expert_ff, width] when gated: gate rows, then up
                                      rows), [experts, width, expert_ff];  DENSE: [expert_ff, width], [width, expert_ff]               */
@@ -573,6 +586,19 @@ typedef struct b200_hybrid_layer_s {
     /* ---- LN_PRE */
     const float *hc1, *hc2;       /* packed [in (streams) | out (streams) | mix (streams x streams, [from][to])], or NULL: x += y     */
     const float *branch_norm;     /* [width] or NULL: RMS norm weight of this mixer's projected result (see B200_NORM_LN_PRE)         */
+    /* ---- RMS_SUM */
+    int in_taps;                  /* taps of the sublayers' input convolution; 0: none                                                */
+    const float *in_conv1, *in_conv2; /* [in_taps, width] (tap-major; the last tap is the current token's): mixer's, feed-forward's   */
+    /* ---- LATENT with q_rank > 0: queries through a normed low-rank row of their own: w_in rows dq (q_rank), then (kv_from < 0) the
+     *      down-projection (kv_rank + rot_dim), then the gate; q = w_uq (rmsnorm(dq) * dq_norm) */
+    int q_rank;
+    int head_gate;                /* 1: ONE gate per head (heads rows) instead of one per value channel                               */
+    const float *dq_norm;         /* [q_rank]                                                                                         */
+    const void *w_uq;             /* [heads*(dim + rot_dim), q_rank]                                                                  */
+    /* ---- MINGRU: heads = dim = 1, vdim = state size; w_in rows z, u, gate (vdim each); b_in [2*vdim] for z and u                   */
+    /* ---- activations with parameters */
+    const float *act_coef;        /* POLYNORM: [4] a, b, c, e                                                                         */
+    float act_limit, act_slope;   /* CLAMP_GLU; act_limit <= 0: no clamp                                                              */
 } b200_hybrid_layer_t;
 
 typedef struct {
@@ -602,7 +628,7 @@ int b200_hybrid_set_scratch(b200_hybrid_t *m, void *ptr, size_t bytes);
  * with a cache of its own [num_pages, B200_KV_PAGE_SIZE, kv_rank + rot_dim] (latent row, then the rotated key part), of the engine dtype
  * (layers may differ in size; each starts 256-byte aligned).  State pool: per recurrent layer fp32 [num_slots, heads, dim, vdim]; DELTA
  * adds the convolutions' last conv - 1 inputs [num_slots, conv - 1, channels], MLSTM the normaliser [num_slots, heads, dim] and the running
- * maximum [num_slots, heads].  A layer that runs several times (loop) owns one such region per run.  Caller-owned. */
+ * maximum [num_slots, heads]; every RMS_SUM layer adds its sublayers' last inputs [num_slots, in_taps - 1, width], one region per sublayer.  A layer that runs several times (loop) owns one such region per run.  Caller-owned. */
 size_t b200_hybrid_kv_pool_bytes(const b200_hybrid_t *m, int num_pages);
 size_t b200_hybrid_state_pool_bytes(const b200_hybrid_t *m, int num_slots);
 int b200_hybrid_set_pools(b200_hybrid_t *m, void *kv_pool, int num_pages, void *state_pool, int num_slots);
@@ -713,6 +739,16 @@ int b200_mlstm_recurrent(const float *rec, float *state, float *n_state, float *
  * unused here) | decay (heads).  state fp32 [num_slots, heads, dim, vdim]; o fp32 [tokens, heads*vdim]. */
 int b200_decay_recurrent(const float *rec, float *state, float *o, const int *seq_start, const int *seq_pos0, const int *seq_slot,
                          int n_seqs, int heads, int kv_heads, int dim, int vdim, b200_stream_t stream);
+
+/* The minGRU recurrence (B200_MIXER_MINGRU).  proj [tokens, ld] of `dtype`: z | u | gate (cols each); bias fp32 [2*cols] for z and u, or
+ * NULL; state fp32 [num_slots, cols]; out [tokens, cols] of `dtype`.  Portions of 8 tokens or more are described by `chunks`, DEVICE int4
+ * {sequence, first packed row, tokens, index in its portion} (a portion's chunks in order and complete; 16-byte aligned); maps: fp32 scratch
+ * [n_chunks, 2, cols].  n_short: tokens in shorter portions.  The other arrays are DEVICE arrays as in b200_hybrid_batch_t. */
+int b200_mingru(const void *proj, int ld, const float *bias, float *state, float *maps, void *out, const int *chunks, int n_chunks,
+                const int *seq_start, const int *seq_pos0, const int *seq_slot, int n_seqs, int n_short, int cols, int dtype,
+                b200_stream_t stream);
+/* In place, row by row: x <- a n(x) + b n(x^2) + c n(x^3) + e, n(v) = v / sqrt(mean over the row of v^2 + eps); coef DEVICE fp32 [4]. */
+int b200_poly_norm(void *x, const float *coef, float eps, int rows, int cols, int dtype, b200_stream_t stream);
 
 /* ========================================== generation loop ========================================= */
 

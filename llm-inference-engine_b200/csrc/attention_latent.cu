@@ -30,7 +30,7 @@ __global__ void __launch_bounds__(128)
 latent_prep_kernel(const T *__restrict__ proj, int ld, int q_col, int kv_col, T *__restrict__ qn, T *__restrict__ qr, T *__restrict__ pool,
                    const float *__restrict__ kv_norm, float eps, const int *__restrict__ tok_seq, const int *__restrict__ tok_pos,
                    const int *__restrict__ block_table, int mpps, int t_pad, int heads, int dim, int rot_dim, int kv_rank, int rot_dims,
-                   float rot_base) {
+                   float rot_base, const T *__restrict__ kv_proj, int kv_ld) {
     extern __shared__ float cs[];  // cos[half] | sin[half]
     __shared__ float red[33];
     const int t = blockIdx.x, half = rot_dims / 2;
@@ -73,7 +73,7 @@ latent_prep_kernel(const T *__restrict__ proj, int ld, int q_col, int kv_col, T 
         }
     }
     if (kv_col < 0) return;  // this layer reads another layer's rows
-    const T *kv = row + kv_col;
+    const T *kv = (kv_proj ? kv_proj + (size_t)t * kv_ld : row) + kv_col;
     float ss = 0.0f;
     for (int c = threadIdx.x; c < kv_rank; c += blockDim.x) {
         const float v = Elem<T>::to_f(kv[c]);
@@ -452,9 +452,31 @@ latent_combine_kernel(const float *__restrict__ part, const int4 *__restrict__ t
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-latent_gate_kernel(const T *__restrict__ ov, const T *__restrict__ gate_in, int gate_ld, T *__restrict__ out, int t_pad, int heads, int vdim) {
+latent_gate_kernel(const T *__restrict__ ov, const T *__restrict__ gate_in, int gate_ld, T *__restrict__ out, int t_pad, int heads, int vdim,
+                   int head_gate) {
     const int t = blockIdx.x;
     constexpr int V = Elem<T>::kVec;
+    if (head_gate) {  // one gate per head
+        const T *gr = gate_in + (size_t)t * gate_ld;
+        if (vdim % V == 0 && ((reinterpret_cast<size_t>(ov) | reinterpret_cast<size_t>(out)) & 15) == 0) {
+            const int pieces = vdim / V;
+            for (int idx = threadIdx.x; idx < heads * pieces; idx += blockDim.x) {
+                const int h = idx / pieces, c = (idx - h * pieces) * V;
+                const float m = 1.0f / (1.0f + expf(-Elem<T>::to_f(gr[h])));
+                float o[V];
+                unpack16<T>(ld_v4(ov + ((size_t)h * t_pad + t) * vdim + c), o);
+#pragma unroll
+                for (int e = 0; e < V; ++e) o[e] *= m;
+                st_v4(out + ((size_t)t * heads + h) * vdim + c, pack16<T>(o));
+            }
+            return;
+        }
+        for (int idx = threadIdx.x; idx < heads * vdim; idx += blockDim.x) {
+            const int h = idx / vdim, c = idx - h * vdim;
+            out[(size_t)t * heads * vdim + idx] = Elem<T>::from_f(Elem<T>::to_f(ov[((size_t)h * t_pad + t) * vdim + c]) / (1.0f + expf(-Elem<T>::to_f(gr[h]))));
+        }
+        return;
+    }
     if (vdim % V == 0 && gate_ld % V == 0 &&
         ((reinterpret_cast<size_t>(ov) | reinterpret_cast<size_t>(gate_in) | reinterpret_cast<size_t>(out)) & 15) == 0) {  // 16-byte pieces
         const int pieces = vdim / V;
@@ -476,14 +498,64 @@ latent_gate_kernel(const T *__restrict__ ov, const T *__restrict__ gate_in, int 
     }
 }
 
+// out[t, :] = in[t, 0 : cols] * rsqrt(mean of squares + eps) * w: the normed low-rank row the queries are projected from.  One warp per row
+template <typename T>
+__global__ void __launch_bounds__(128)
+rms_rows_kernel(const T *__restrict__ in, int ld, const float *__restrict__ w, float eps, T *__restrict__ out, int tokens, int cols) {
+    const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (t >= tokens) return;
+    constexpr int V = Elem<T>::kVec;
+    const T *row = in + (size_t)t * ld;
+    T *dst = out + (size_t)t * cols;
+    const bool vec = cols % V == 0 && ld % V == 0 && ((reinterpret_cast<size_t>(in) | reinterpret_cast<size_t>(out) | reinterpret_cast<size_t>(w)) & 15) == 0;
+    float ss = 0.0f;
+    if (vec) {
+#pragma unroll 4
+        for (int c = lane * V; c < cols; c += 32 * V) {
+            float f[V];
+            unpack16<T>(ld_v4(row + c), f);
+#pragma unroll
+            for (int i = 0; i < V; ++i) ss = fmaf(f[i], f[i], ss);
+        }
+    } else {
+        for (int c = lane; c < cols; c += 32) {
+            const float f = Elem<T>::to_f(row[c]);
+            ss = fmaf(f, f, ss);
+        }
+    }
+    const float inv = rsqrtf(warp_sum(ss) / (float)cols + eps);
+    if (vec) {
+#pragma unroll 4
+        for (int c = lane * V; c < cols; c += 32 * V) {
+            float f[V];
+            unpack16<T>(ld_v4(row + c), f);
+#pragma unroll
+            for (int i = 0; i < V; i += 4) {
+                const float4 g = *reinterpret_cast<const float4 *>(w + c + i);
+                f[i] *= inv * g.x, f[i + 1] *= inv * g.y, f[i + 2] *= inv * g.z, f[i + 3] *= inv * g.w;
+            }
+            st_v4(dst + c, pack16<T>(f));
+        }
+        return;
+    }
+    for (int c = lane; c < cols; c += 32) dst[c] = Elem<T>::from_f(Elem<T>::to_f(row[c]) * inv * w[c]);
+}
+
+int launch_rms_rows(int dtype, const void *in, int ld, const float *w, float eps, void *out, int tokens, int cols, cudaStream_t st) {
+    if (tokens == 0) return B200_OK;
+    B200_DISPATCH_DTYPE(dtype, { rms_rows_kernel<T><<<(tokens + 3) / 4, 128, 0, st>>>((const T *)in, ld, w, eps, (T *)out, tokens, cols); });
+    return cuda_status("rms_rows launch");
+}
+
 int launch_latent_prep(int dtype, const void *proj, int ld, int q_col, int kv_col, void *qn, void *qr, void *pool, const float *kv_norm,
                        float eps, const int *tok_seq, const int *tok_pos, const int *block_table, int mpps, int tokens, int t_pad, int heads,
-                       int dim, int rot_dim, int kv_rank, int rot_dims, float rot_base, cudaStream_t st) {
+                       int dim, int rot_dim, int kv_rank, int rot_dims, float rot_base, cudaStream_t st, const void *kv_proj, int kv_ld) {
     if (tokens == 0) return B200_OK;
     const size_t smem = (size_t)std::max(rot_dims, 2) * sizeof(float);
     B200_DISPATCH_DTYPE(dtype, {
         latent_prep_kernel<T><<<tokens, 128, smem, st>>>((const T *)proj, ld, q_col, kv_col, (T *)qn, (T *)qr, (T *)pool, kv_norm, eps, tok_seq,
-                                                        tok_pos, block_table, mpps, t_pad, heads, dim, rot_dim, kv_rank, rot_dims, rot_base);
+                                                        tok_pos, block_table, mpps, t_pad, heads, dim, rot_dim, kv_rank, rot_dims, rot_base,
+                                                        (const T *)kv_proj, kv_ld);
     });
     return cuda_status("latent_prep launch");
 }
@@ -577,10 +649,10 @@ int launch_latent_attention_tiles(int dtype, const void *ql, const void *qr, con
 }
 
 int launch_latent_gate(int dtype, const void *ov, const void *gate_in, int gate_ld, void *out, int tokens, int t_pad, int heads, int vdim,
-                       cudaStream_t st) {
+                       cudaStream_t st, int head_gate) {
     if (tokens == 0) return B200_OK;
     B200_DISPATCH_DTYPE(dtype, {
-        latent_gate_kernel<T><<<tokens, 256, 0, st>>>((const T *)ov, (const T *)gate_in, gate_ld, (T *)out, t_pad, heads, vdim);
+        latent_gate_kernel<T><<<tokens, 256, 0, st>>>((const T *)ov, (const T *)gate_in, gate_ld, (T *)out, t_pad, heads, vdim, head_gate);
     });
     return cuda_status("latent_gate launch");
 }

@@ -20,6 +20,10 @@
 // mixers side by side arrive as two projected rows, each RMS-normed over the width) and leaves the next sublayer's layer-normed input:
 //   input projection -> mixer (scored attention | delta rule | state-space | linear attention; a second mixer beside it) -> output
 //   projection(s) -> streams + next norm;  gate|up projection -> act(gate) * up -> down projection -> streams + next norm
+// Layers whose norm takes the sum (B200_NORM_RMS_SUM: x <- rmsnorm(alpha x + sublayer(x + conv(x))) * g; sum_norm.cu) run in the same loop as
+// the post-norm ones; the convolved input of a sublayer comes from the kernel that writes x (decode batches) or from one that follows it:
+//   minGRU mixer:     input projection -> affine-map scan over chunks (or one step per decoded token) -> output projection
+//   latent mixer, q_rank > 0: down-projections -> row norm -> query up-projection -> as above, one gate per head
 // and at the end: final norm of the wanted rows -> LM head with fp32 logits (scaled, soft-capped).
 // Everything is stream-ordered and allocation-free; the only host->device traffic of a call is one copy of the batch description.
 #include "hybrid_ops.cuh"
@@ -679,6 +683,7 @@ struct LayerPlan : MixerPlan {
     int n_in = 0;                     // rows of the fused input projection
     int layer = 0;                    // which layer this run executes
     int entry = -1;                   // >= 0: the run opens pass `entry` of the looped block (the entry step comes first)
+    size_t conv_off[2] = {0, 0};      // RMS_SUM: rings of the mixer's and the feed-forward's input convolution in the state pool
     MixerPlan side;                   // the second mixer beside the first
 };
 
@@ -750,7 +755,9 @@ int n_in_of(const b200_hybrid_layer_t &l) {
     if (l.norm == B200_NORM_LN_PARALLEL) return mixer_rows(l) + (l.side ? mixer_rows(*l.side) : 0) + (l.mlp == B200_MLP_DENSE ? 2 * l.expert_ff : 0);
     if (l.norm == B200_NORM_LN_PRE) return mixer_rows(l) + (l.side ? mixer_rows(*l.side) : 0);
     if (l.mixer == B200_MIXER_ATTN_CHUNKED) return (2 * l.heads + l.kv_heads) * l.dim;
-    if (l.mixer == B200_MIXER_LATENT) return l.heads * (l.dim + l.rot_dim) + l.heads * l.vdim + (l.kv_from < 0 ? l.kv_rank + l.rot_dim : 0);
+    if (l.mixer == B200_MIXER_LATENT)
+        return (l.q_rank > 0 ? l.q_rank : l.heads * (l.dim + l.rot_dim)) + (l.head_gate ? l.heads : l.heads * l.vdim) + (l.kv_from < 0 ? l.kv_rank + l.rot_dim : 0);
+    if (l.mixer == B200_MIXER_MINGRU) return 3 * l.vdim;
     return 2 * l.heads * l.dim + 2 * l.heads * l.vdim + l.decay_rank;
 }
 
@@ -784,6 +791,7 @@ Carve carve(const b200_hybrid *m) {
             lqn = std::max(lqn, (size_t)l.heads * t_pad * l.dim), lqr = std::max(lqr, T * l.heads * l.rot_dim);
             lql = std::max(lql, (size_t)l.heads * t_pad * l.kv_rank), lov = std::max(lov, (size_t)l.heads * t_pad * l.vdim);
             lheads = std::max(lheads, (size_t)l.heads);
+            if (l.q_rank > 0) n_mix = std::max(n_mix, (size_t)std::max(l.q_rank, l.heads * (l.dim + l.rot_dim)));  // normed row (mix2), queries (mix)
             lpart = std::max(lpart, (size_t)kLatentPartTiles * l.heads * (l.kv_rank + 2));
         }
         const size_t g = l.gated ? 3 : 1;  // gated: [gate | up] and the product beside it
@@ -814,9 +822,10 @@ Carve carve(const b200_hybrid *m) {
     k.lpart = align256(lpart * 4);
     // meta: attention tiles [4 * (T/64 + S), padded] | ids | tok_seq | tok_pos | want | short-portion token list [T each] | seq_start [S+1] |
     //       pos0 | slot [S each] | block table [S * mpps]
+    //       | chunks of the minGRU mixer [4 * (T/64 + S)]
     //       | latent mixers: one-token tiles of the short portions [4 * T] | head of every row tile of 64 and of 128 [heads * t_pad / 64,
     //         heads * t_pad / 128] | live row tiles per layer, of 64 and of 128 [layers each]
-    k.meta = align256((4 * (T / 64 + (size_t)c.max_seqs + 1) + 5 * T + 3 * (size_t)c.max_seqs + 1 + (size_t)c.max_seqs * c.max_pages_per_seq +
+    k.meta = align256((8 * (T / 64 + (size_t)c.max_seqs + 1) + 5 * T + 3 * (size_t)c.max_seqs + 1 + (size_t)c.max_seqs * c.max_pages_per_seq +
                        (lheads ? 4 * T : 0) + 2 * lheads * (t_pad / 64) + 2 * (size_t)c.num_layers) * 4);
     // moe ints: sel_expert | pair_row [T*top each] | row_token [rows] | tile_expert [rows / tile] | n_tiles
     k.moe_i = align256((2 * T * top + rows + rows / kMoeTileM + 4) * 4);
@@ -908,8 +917,8 @@ static int check_scored_mixer(const b200_hybrid_layer_t *w) {
 int b200_hybrid_set_layer(b200_hybrid_t *m, int layer, const b200_hybrid_layer_t *w) {
     B200_REQUIRE(m && w, "hybrid_set_layer: null argument");
     B200_REQUIRE(layer >= 0 && layer < m->cfg.num_layers, "hybrid_set_layer: layer %d outside [0, %d)", layer, m->cfg.num_layers);
-    B200_REQUIRE(w->mixer >= B200_MIXER_ATTN_CHUNKED && w->mixer <= B200_MIXER_LINEAR, "hybrid_set_layer: unknown mixer kind %d", w->mixer);
-    B200_REQUIRE(w->norm >= B200_NORM_RMS_POST && w->norm <= B200_NORM_LN_PRE, "hybrid_set_layer: unknown norm kind %d", w->norm);
+    B200_REQUIRE(w->mixer >= B200_MIXER_ATTN_CHUNKED && w->mixer <= B200_MIXER_MINGRU, "hybrid_set_layer: unknown mixer kind %d", w->mixer);
+    B200_REQUIRE(w->norm >= B200_NORM_RMS_POST && w->norm <= B200_NORM_RMS_SUM, "hybrid_set_layer: unknown norm kind %d", w->norm);
     B200_REQUIRE(w->heads > 0 && w->dim > 0 && w->w_in && w->w_out, "hybrid_set_layer: mixer sizes / weights missing");
     if (w->norm == B200_NORM_LN_PARALLEL || w->norm == B200_NORM_LN_PRE) {
         // LN_PARALLEL: one norm, one input projection, one output projection; the mixers are of the kinds that read a shared projection
@@ -942,11 +951,17 @@ int b200_hybrid_set_layer(b200_hybrid_t *m, int layer, const b200_hybrid_layer_t
         m->scratch = nullptr;
         return B200_OK;
     }
-    B200_REQUIRE(w->mixer <= B200_MIXER_LATENT && !w->side, "hybrid_set_layer: mixer kind %d needs the shared-norm or the pre-norm layer form", w->mixer);
+    B200_REQUIRE((w->mixer <= B200_MIXER_LATENT || w->mixer == B200_MIXER_MINGRU) && !w->side, "hybrid_set_layer: mixer kind %d needs the shared-norm or the pre-norm layer form", w->mixer);
     B200_REQUIRE(m->cfg.loop_times == 0, "hybrid_set_layer: only shared-norm and pre-norm layers can be looped");
-    if (w->norm == B200_NORM_RMS_POST) B200_REQUIRE(w->norm1, "hybrid_set_layer: norm weight missing");
+    const bool sum = w->norm == B200_NORM_RMS_SUM;
+    if (w->norm == B200_NORM_RMS_POST || sum) B200_REQUIRE(w->norm1, "hybrid_set_layer: norm weight missing");
     else B200_REQUIRE(w->pre1 && w->post1, "hybrid_set_layer: norm parameters missing");
-    if (w->mixer == B200_MIXER_ATTN_CHUNKED) {
+    if (sum) B200_REQUIRE(w->in_taps >= 0 && w->in_taps <= 64 && (w->in_taps == 0 || (w->in_conv1 && (w->mlp == B200_MLP_NONE || w->in_conv2))),
+                          "hybrid_set_layer: input convolution of %d taps (at most 64) / its weights", w->in_taps);
+    else B200_REQUIRE(w->in_taps == 0, "hybrid_set_layer: only layers whose norm takes the sum have an input convolution");
+    if (w->mixer == B200_MIXER_MINGRU) {
+        B200_REQUIRE(w->heads == 1 && w->dim == 1 && w->vdim > 0, "hybrid_set_layer: the minGRU's state size is vdim, with one head of dim 1");
+    } else if (w->mixer == B200_MIXER_ATTN_CHUNKED) {
         B200_REQUIRE(w->kv_heads > 0 && w->heads % w->kv_heads == 0, "hybrid_set_layer: heads %d not a multiple of kv_heads %d", w->heads, w->kv_heads);
         B200_REQUIRE(w->vdim == w->dim, "hybrid_set_layer: this attention's values are its keys: vdim %d must equal dim %d", w->vdim, w->dim);
         B200_REQUIRE(w->chunk >= 0, "hybrid_set_layer: negative chunk");
@@ -957,23 +972,28 @@ int b200_hybrid_set_layer(b200_hybrid_t *m, int layer, const b200_hybrid_layer_t
         B200_REQUIRE(w->w_uk_t && w->w_uv, "hybrid_set_layer: latent attention up-projections missing");
         B200_REQUIRE(w->kv_from < layer, "hybrid_set_layer: layer %d cannot read the latent rows of layer %d", layer, w->kv_from);
         B200_REQUIRE(w->kv_from >= 0 || w->kv_norm, "hybrid_set_layer: latent row norm weight missing");
+        B200_REQUIRE(w->q_rank >= 0 && (w->q_rank == 0 || (w->dq_norm && w->w_uq)), "hybrid_set_layer: the low-rank query's norm / up-projection missing");
     } else {
         B200_REQUIRE(w->vdim > 0 && w->decay_rank > 0 && w->tau > 0.0f && w->w_decay && w->out_norm, "hybrid_set_layer: gla sizes / weights missing");
     }
     B200_REQUIRE(w->mlp == B200_MLP_NONE || w->mlp == B200_MLP_MOE || w->mlp == B200_MLP_DENSE, "hybrid_set_layer: unknown feed-forward kind %d", w->mlp);
     if (w->mlp != B200_MLP_NONE) {
-        if (w->norm == B200_NORM_RMS_POST) B200_REQUIRE(w->norm2, "hybrid_set_layer: feed-forward norm weight missing");
+        if (w->norm == B200_NORM_RMS_POST || sum) B200_REQUIRE(w->norm2, "hybrid_set_layer: feed-forward norm weight missing");
         else B200_REQUIRE(w->pre2 && w->post2, "hybrid_set_layer: feed-forward norm parameters missing");
-        B200_REQUIRE(w->act >= B200_ACT_RELU2 && w->act <= B200_ACT_RELU, "hybrid_set_layer: unknown activation %d", w->act);
+        B200_REQUIRE(w->act >= B200_ACT_RELU2 && w->act <= B200_ACT_CLAMP_GLU, "hybrid_set_layer: unknown activation %d", w->act);
+        if (w->act == B200_ACT_POLYNORM)
+            B200_REQUIRE(w->mlp == B200_MLP_DENSE && !w->gated && !w->b_up && w->act_coef, "hybrid_set_layer: the polynomial of norms is the activation of a dense, not gated feed-forward without bias");
+        if (w->act == B200_ACT_CLAMP_GLU) B200_REQUIRE(w->gated, "hybrid_set_layer: the clamped gate is the activation of gated feed-forwards");
         B200_REQUIRE(w->expert_ff > 0 && w->w_up && w->w_down, "hybrid_set_layer: feed-forward sizes / weights missing");
     }
     if (w->mlp == B200_MLP_MOE) {
         B200_REQUIRE(w->experts > 0 && w->top > 0 && w->shared_ff >= 0 && w->identity >= 0, "hybrid_set_layer: bad expert counts");
         B200_REQUIRE(w->route == B200_ROUTE_SIGMOID || w->route == B200_ROUTE_SOFTMAX, "hybrid_set_layer: unknown router kind %d", w->route);
         if (w->route == B200_ROUTE_SIGMOID) {
-            B200_REQUIRE(w->top <= w->experts && w->identity == 0 && !w->gated, "hybrid_set_layer: the sigmoid router has no identity or gated experts");
-            B200_REQUIRE(w->norm == B200_NORM_RMS_POST, "hybrid_set_layer: the sigmoid router weighs the fp32 residual row: post-norm layers only");
+            B200_REQUIRE(w->top <= w->experts && w->identity == 0, "hybrid_set_layer: the sigmoid router has no identity experts");
+            B200_REQUIRE(w->norm == B200_NORM_RMS_POST || sum, "hybrid_set_layer: the sigmoid router's weights go on the experts' inputs: post-norm layers only");
         } else {
+            B200_REQUIRE(!sum, "hybrid_set_layer: layers whose norm takes the sum route by sigmoid scores");
             B200_REQUIRE(w->top <= w->experts + w->identity, "hybrid_set_layer: top %d of %d router outputs", w->top, w->experts + w->identity);
         }
         B200_REQUIRE(w->w_router, "hybrid_set_layer: router weights missing");
@@ -1065,6 +1085,14 @@ void place_mixer(const b200_hybrid_layer_t &l, size_t es, int num_pages, int num
     }
     if (plan) *plan = p;
 }
+// the rings of an RMS_SUM layer's input convolutions
+void place_conv(const b200_hybrid_layer_t &l, int width, int num_slots, size_t &stt, size_t *off) {
+    if (l.norm != B200_NORM_RMS_SUM || l.in_taps < 2) return;
+    for (int k = 0; k < (l.mlp == B200_MLP_NONE ? 1 : 2); ++k) {
+        if (off) off[k] = stt;
+        stt += align256((size_t)num_slots * (l.in_taps - 1) * width * 4);
+    }
+}
 }  // namespace
 
 size_t b200_hybrid_kv_pool_bytes(const b200_hybrid_t *m, int num_pages) {
@@ -1086,6 +1114,7 @@ size_t b200_hybrid_state_pool_bytes(const b200_hybrid_t *m, int num_slots) {
         if (!m->layer_set[lp.layer]) continue;
         place_mixer(m->layers[lp.layer], 2, 1, num_slots, kv, stt, nullptr);
         if (m->layers[lp.layer].side) place_mixer(*m->layers[lp.layer].side, 2, 1, num_slots, kv, stt, nullptr);
+        place_conv(m->layers[lp.layer], m->cfg.width, num_slots, stt, nullptr);
     }
     return stt ? stt : 256;
 }
@@ -1102,6 +1131,7 @@ int b200_hybrid_set_pools(b200_hybrid_t *m, void *kv_pool, int num_pages, void *
         const b200_hybrid_layer_t &l = m->layers[i];
         place_mixer(l, es, num_pages, num_slots, kv, stt, &lp);
         if (l.side) place_mixer(*l.side, es, num_pages, num_slots, kv, stt, &lp.side);
+        place_conv(l, m->cfg.width, num_slots, stt, lp.conv_off);
         if (l.mixer == B200_MIXER_LATENT && l.kv_from >= 0) {  // the rows of an earlier layer, which must own them and rotate them alike
             const b200_hybrid_layer_t &o = m->layers[l.kv_from];
             B200_REQUIRE(o.mixer == B200_MIXER_LATENT && o.kv_from < 0 && o.kv_rank == l.kv_rank && o.rot_dim == l.rot_dim &&
@@ -1144,9 +1174,11 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
     const bool lat_tc = c.dtype != B200_F32 && NT >= 256;
     const int t_pad = lat_tc ? (NT + 127) / 128 * 128 : (NT + kMoeTileM - 1) / kMoeTileM * kMoeTileM;
     const int tph = t_pad / kMoeTileM, tph128 = lat_tc ? t_pad / 128 : 0;
-    const size_t n_tile_ints = 4 * ((size_t)NT / 64 + S + 1), n_stile_ints = lat_by_head ? (size_t)4 * NT : 0;
-    hm.assign(n_tile_ints + n_stile_ints + (size_t)5 * NT + 3 * S + 1 + (size_t)S * mpps + (size_t)lat_heads * (tph + tph128) + 2 * c.num_layers, 0);
-    int *h_tiles = hm.data(), *h_stiles = h_tiles + n_tile_ints, *h_ids = h_stiles + n_stile_ints, *h_seq = h_ids + NT, *h_pos = h_seq + NT,
+    bool any_mingru = false;
+    for (int i = 0; i < c.num_layers; ++i) any_mingru |= m->layers[i].mixer == B200_MIXER_MINGRU;
+    const size_t n_tile_ints = 4 * ((size_t)NT / 64 + S + 1), n_chunk_ints = any_mingru ? n_tile_ints : 0, n_stile_ints = lat_by_head ? (size_t)4 * NT : 0;
+    hm.assign(n_tile_ints + n_chunk_ints + n_stile_ints + (size_t)5 * NT + 3 * S + 1 + (size_t)S * mpps + (size_t)lat_heads * (tph + tph128) + 2 * c.num_layers, 0);
+    int *h_tiles = hm.data(), *h_chunks = h_tiles + n_tile_ints, *h_stiles = h_chunks + n_chunk_ints, *h_ids = h_stiles + n_stile_ints, *h_seq = h_ids + NT, *h_pos = h_seq + NT,
         *h_want = h_pos + NT, *h_short = h_want + NT, *h_start = h_short + NT, *h_pos0 = h_start + S + 1, *h_slot = h_pos0 + S, *h_bt = h_slot + S,
         *h_lat_head = h_bt + (size_t)S * mpps, *h_lat_head128 = h_lat_head + (size_t)lat_heads * tph,
         *h_lat_n = h_lat_head128 + (size_t)lat_heads * tph128, *h_lat_n128 = h_lat_n + c.num_layers;
@@ -1158,7 +1190,12 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
     }
     // prompt portions go to the tensor-core attention in tiles of <= 64 consecutive tokens, short ones (decoded tokens) to the per-token kernel
     constexpr int kShortPortion = 8;
-    int n_tiles = 0, n_short = 0, gla_kinds = 0;
+    static_assert(kShortPortion == kMingruShort, "one list of short portions serves both");
+    int n_tiles = 0, n_short = 0, n_chunks = 0, gla_kinds = 0;
+    // minGRU chunks: at most 64 per portion (a chunk composes the maps of all chunks before it), of whole multiples of 64 tokens
+    int longest = 0;
+    for (int s = 0; s < S; ++s) longest = std::max(longest, b->seq_start[s + 1] - b->seq_start[s]);
+    const int chunk_tokens = std::max(1, (longest + 4095) / 4096) * 64;
     for (int s = 0; s < S; ++s) {
         const int t0 = b->seq_start[s], t1 = b->seq_start[s + 1];
         gla_kinds |= t1 - t0 == 1 ? kGlaOneToken : (t1 - t0 > 1 ? kGlaManyTokens : 0);
@@ -1185,6 +1222,11 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
                 int *tl = h_tiles + 4 * n_tiles;
                 tl[0] = s, tl[1] = t, tl[2] = std::min(64, t1 - t), tl[3] = h_pos[t];
             }
+            if (any_mingru)
+                for (int t = t0; t < t1; t += chunk_tokens, ++n_chunks) {
+                    int *ch = h_chunks + 4 * n_chunks;
+                    ch[0] = s, ch[1] = t, ch[2] = std::min(chunk_tokens, t1 - t), ch[3] = (t - t0) / chunk_tokens;
+                }
         }
         h_start[s] = t0, h_pos0[s] = b->seq_pos0[s], h_slot[s] = b->seq_slot[s];
         for (int p = 0; p < mpps; ++p) h_bt[(size_t)s * mpps + p] = b->block_table[(size_t)s * mpps + p];
@@ -1201,7 +1243,7 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
     cudaStream_t st = as_stream(stream);
     NvtxRange range("hybrid_forward");
     if (cudaMemcpyAsync(m->meta, hm.data(), hm.size() * sizeof(int), cudaMemcpyHostToDevice, st) != cudaSuccess) return cuda_status("hybrid_forward meta copy");
-    const int *d_tiles = m->meta, *d_stiles = d_tiles + n_tile_ints, *d_ids = d_stiles + n_stile_ints, *d_seq = d_ids + NT, *d_pos = d_seq + NT,
+    const int *d_tiles = m->meta, *d_chunks = d_tiles + n_tile_ints, *d_stiles = d_chunks + n_chunk_ints, *d_ids = d_stiles + n_stile_ints, *d_seq = d_ids + NT, *d_pos = d_seq + NT,
               *d_want = d_pos + NT, *d_short = d_want + NT, *d_start = d_short + NT, *d_pos0 = d_start + S + 1, *d_slot = d_pos0 + S, *d_bt = d_slot + S,
               *d_lat_head = d_bt + (size_t)S * mpps, *d_lat_head128 = d_lat_head + (size_t)lat_heads * tph,
               *d_lat_n = d_lat_head128 + (size_t)lat_heads * tph128, *d_lat_n128 = d_lat_n + c.num_layers;
@@ -1218,9 +1260,11 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
     const int n_runs = (int)m->plan.size();
     const bool shared_norm = m->layers[0].norm == B200_NORM_LN_PARALLEL;  // layers of one norm whose sublayers share the projections
     const bool pre_norm = m->layers[0].norm == B200_NORM_LN_PRE;          // pre-norm layers on residual streams
+    const bool sum_norm = m->layers[0].norm == B200_NORM_RMS_SUM;         // layers whose norm takes the sum
     for (int i = 0; i < c.num_layers; ++i)
-        B200_REQUIRE((m->layers[i].norm == B200_NORM_LN_PARALLEL) == shared_norm && (m->layers[i].norm == B200_NORM_LN_PRE) == pre_norm,
-                     "hybrid_forward: shared-norm layers, pre-norm layers and others do not mix in one model");
+        B200_REQUIRE((m->layers[i].norm == B200_NORM_LN_PARALLEL) == shared_norm && (m->layers[i].norm == B200_NORM_LN_PRE) == pre_norm &&
+                         (m->layers[i].norm == B200_NORM_RMS_SUM) == sum_norm,
+                     "hybrid_forward: shared-norm layers, pre-norm layers, layers whose norm takes the sum and others do not mix in one model");
     if (shared_norm && c.loop_times > 0 && (!m->w_entry || !m->loop_step)) {
         set_error("hybrid_forward: the looped block's entry weights are not set");
         return B200_ERR_STATE;
@@ -1250,7 +1294,7 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
         B200_DISPATCH_DTYPE(dt, {
             embed_rows_kernel<T><<<NT, 128, 0, st>>>(d_ids, (const T *)m->embedding, m->x, (T *)nullptr, 0, width, c.vocab, c.embed_scale != 0.0f ? c.embed_scale : 1.0f);
         });
-    } else {
+    } else if (!sum_norm) {
     B200_DISPATCH_DTYPE(dt, { embed_f32_kernel<T><<<NT, 128, 0, st>>>(d_ids, (const T *)m->embedding, m->x, f32 ? nullptr : (T *)m->h, width, c.vocab,
                                                                       c.embed_scale != 0.0f ? c.embed_scale : 1.0f); });
     }
@@ -1414,6 +1458,35 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
         return hand_over(run + 1, m->y, l.b_out, layer_trace ? layer_trace + (size_t)run * NT * width : nullptr);
     };
 
+    // ---- layers whose norm takes the sum: the input convolution of sublayer `sub` (0: mixer, 1: feed-forward) of layer li
+    const PortionMap pm = {d_seq, d_pos, d_start, d_pos0, d_slot};
+    const int one_token = gla_kinds == kGlaOneToken;
+    auto ring_conv = [&](int li, int sub) -> RingConv {
+        const b200_hybrid_layer_t &l = m->layers[li];
+        RingConv r;
+        r.taps = l.in_taps, r.w = sub ? l.in_conv2 : l.in_conv1;
+        if (l.in_taps > 1) r.ring = (float *)(m->state_pool + m->plan[li].conv_off[sub]);
+        return r;
+    };
+    auto conv_input = [&](const RingConv &cv) -> int {  // m->h = the coming sublayer's input, unless the kernel that wrote x has formed it
+        return one_token || cv.taps == 0 ? B200_OK : launch_conv_input(dt, m->x, m->h, width, cv, pm, NT, st);
+    };
+    // x <- rmsnorm(alpha * x + result of sublayer `sub` of layer li) * g, and the input of the sublayer that follows
+    auto sum_step = [&](int li, int sub, const void *y_dense, const void *y_rows, const int *pair_row, const void *y_shared, const float *gate,
+                        float *trace) -> int {
+        const b200_hybrid_layer_t &l = m->layers[li];
+        const bool ff_next = sub == 0 && l.mlp != B200_MLP_NONE, more = ff_next || li + 1 < c.num_layers;
+        const RingConv next = more ? (ff_next ? ring_conv(li, 1) : ring_conv(li + 1, 0)) : RingConv();
+        RUN(launch_sum_norm(dt, m->x, y_dense, y_rows, pair_row, l.top, y_shared, gate, c.residual_scale,
+                            sub ? l.norm2 : l.norm1, c.norm_eps, width, trace, more ? m->h : nullptr, ring_conv(li, sub), next, one_token, pm, NT, st));
+        return more ? conv_input(next) : B200_OK;
+    };
+    if (sum_norm) {
+        RUN(launch_embed_pos(dt, d_ids, m->embedding, m->x, m->h, width, c.vocab, c.embed_scale != 0.0f ? c.embed_scale : 1.0f, c.pos_base, ring_conv(0, 0),
+                             one_token, pm, NT, st));
+        RUN(conv_input(ring_conv(0, 0)));
+    }
+
     auto cast_x = [&]() -> const void * { return f32 ? (const void *)m->x : (const void *)m->h; };
     auto postnorm = [&](const void *y_dense, const void *y_rows, const int *pair_row, int top, const void *y_shared, const float *gate,
                         const float *g, float *trace) -> int {
@@ -1462,7 +1535,7 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
         const bool dyt = l.norm == B200_NORM_DYT_PRE_POST;
         float *trace = (layer_trace && l.mlp == B200_MLP_NONE) ? layer_trace + (size_t)li * NT * width : nullptr;
         if (dyt && !h_normed) RUN(residual(false, nullptr, nullptr, nullptr, nullptr, nullptr, 0, nullptr, nullptr, l.norm, nullptr, nullptr, l.pre1, nullptr));
-        const void *h = dyt ? (const void *)m->h : cast_x();
+        const void *h = dyt || sum_norm ? (const void *)m->h : cast_x();
         RUN(linear(m, h, l.w_in, m->proj, NT, width, lp.n_in, st));
         int n_mixed = 0;  // columns of the mixer's result before the output projection
         if (l.mixer == B200_MIXER_ATTN_CHUNKED) {
@@ -1483,10 +1556,17 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
             n_mixed = hd;
         } else if (l.mixer == B200_MIXER_LATENT) {
             const int nq = l.heads * (l.dim + l.rot_dim), hv = l.heads * l.vdim;
-            const char *gate = (const char *)m->proj + (size_t)nq * es;
+            const bool low_q = l.q_rank > 0;
+            const int gate_col = low_q ? l.q_rank + (l.kv_from < 0 ? l.kv_rank + l.rot_dim : 0) : nq;
+            const char *gate = (const char *)m->proj + (size_t)gate_col * es;
             char *pool = m->kv_pool + lp.k_off;
-            RUN(launch_latent_prep(dt, m->proj, lp.n_in, 0, l.kv_from < 0 ? nq + hv : -1, m->lqn, m->lqr, pool, l.kv_norm, c.norm_eps, d_seq, d_pos, d_bt,
-                                   mpps, NT, t_pad, l.heads, l.dim, l.rot_dim, l.kv_rank, l.rot_dims, l.rot_base, st));
+            if (low_q) {  // the queries come through a normed low-rank row
+                RUN(launch_rms_rows(dt, m->proj, lp.n_in, l.dq_norm, c.norm_eps, m->mix2, NT, l.q_rank, st));
+                RUN(linear(m, m->mix2, l.w_uq, m->mix, NT, l.q_rank, nq, st));
+            }
+            const int kv_col = l.kv_from >= 0 ? -1 : (low_q ? l.q_rank : nq + (l.head_gate ? l.heads : hv));
+            RUN(launch_latent_prep(dt, low_q ? m->mix : m->proj, low_q ? nq : lp.n_in, 0, kv_col, m->lqn, m->lqr, pool, l.kv_norm, c.norm_eps, d_seq, d_pos,
+                                   d_bt, mpps, NT, t_pad, l.heads, l.dim, l.rot_dim, l.kv_rank, l.rot_dims, l.rot_base, st, low_q ? m->proj : nullptr, lp.n_in));
             // the per-head products: rows past the batch's tokens hold whatever the scratch held; a row of a product depends on its own
             // input row only and those rows are never read
             auto head_product = [&](const void *a, const void *w, void *out, int N, int K) -> int {
@@ -1514,8 +1594,12 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
                                             l.scale, l.window, max_keys, st));
             }
             RUN(head_product(m->lol, l.w_uv, m->lov, l.vdim, l.kv_rank));  // out[h] = (sum_j p c_j) . W_uv,h^T
-            RUN(launch_latent_gate(dt, m->lov, gate, lp.n_in, m->mix2, NT, t_pad, l.heads, l.vdim, st));
+            RUN(launch_latent_gate(dt, m->lov, gate, lp.n_in, m->mix2, NT, t_pad, l.heads, l.vdim, st, l.head_gate));
             n_mixed = hv;
+        } else if (l.mixer == B200_MIXER_MINGRU) {
+            RUN(launch_mingru(dt, m->proj, lp.n_in, l.b_in, (float *)(m->state_pool + lp.state_off), m->f32a, m->mix2, d_chunks, n_chunks, d_start, d_pos0,
+                              d_slot, S, n_short, l.vdim, st));
+            n_mixed = l.vdim;
         } else {
             const int hd = l.heads * l.dim, hv = l.heads * l.vdim;
             const char *gate = (const char *)m->proj + (size_t)(2 * hd + hv) * es;
@@ -1526,7 +1610,9 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
             n_mixed = hv;
         }
         RUN(linear(m, m->mix2, l.w_out, m->y, NT, n_mixed, width, st));
-        if (dyt) {
+        if (sum_norm) {
+            RUN(sum_step(li, 0, m->y, nullptr, nullptr, nullptr, nullptr, trace));
+        } else if (dyt) {
             const float *pre = next_pre(li, 0);
             RUN(residual(true, m->y, nullptr, nullptr, nullptr, nullptr, 0, nullptr, nullptr, l.norm, l.post1, l.ls1, pre, trace));
             h_normed = pre != nullptr;
@@ -1536,7 +1622,7 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
         }
         if (l.mlp == B200_MLP_NONE) continue;
         trace = layer_trace ? layer_trace + (size_t)li * NT * width : nullptr;
-        const void *h2 = dyt ? (const void *)m->h : cast_x();
+        const void *h2 = dyt || sum_norm ? (const void *)m->h : cast_x();
         const float *pre = next_pre(li, 1);
         const int inner_cols = l.gated ? 2 : 1;
         if (l.mlp == B200_MLP_DENSE) {
@@ -1545,19 +1631,24 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
             if (l.gated) {
                 act = up + (size_t)NT * 2 * l.expert_ff * es;
                 if (l.b_up) RUN(launch_bias_activation(dt, up, l.b_up, NT, 2 * l.expert_ff, -1, st));
-                RUN(launch_gated_activation(dt, up, act, NT, l.expert_ff, l.act, nullptr, 0, st));
+                RUN(launch_gated_activation(dt, up, act, NT, l.expert_ff, l.act, nullptr, 0, st, l.act_limit, l.act_slope));
+            } else if (l.act == B200_ACT_POLYNORM) {
+                RUN(launch_poly_norm(dt, up, l.act_coef, c.norm_eps, NT, l.expert_ff, st));
             } else {
                 RUN(launch_bias_activation(dt, up, l.b_up, NT, l.expert_ff, l.act, st));
             }
             RUN(linear(m, act, l.w_down, m->ys, NT, l.expert_ff, width, st));
-            if (dyt) RUN(residual(true, m->ys, l.b_down, nullptr, nullptr, nullptr, 0, nullptr, nullptr, l.norm, l.post2, l.ls2, pre, trace));
+            if (sum_norm) {
+                if (l.b_down) RUN(launch_bias_activation(dt, m->ys, l.b_down, NT, width, -1, st));
+                RUN(sum_step(li, 1, m->ys, nullptr, nullptr, nullptr, nullptr, trace));
+            } else if (dyt) RUN(residual(true, m->ys, l.b_down, nullptr, nullptr, nullptr, 0, nullptr, nullptr, l.norm, l.post2, l.ls2, pre, trace));
             else RUN(residual(true, m->ys, l.b_down, nullptr, nullptr, nullptr, 0, nullptr, nullptr, l.norm, l.norm2, nullptr, nullptr, trace));
             h_normed = dyt && pre != nullptr;
             continue;
         }
         const int pairs = NT * l.top;
         const bool softmax = l.route == B200_ROUTE_SOFTMAX;
-        const int outputs = softmax ? l.experts + l.identity : l.experts + 1;
+        const int outputs = softmax ? l.experts + l.identity : l.experts + (l.shared_ff > 0 ? 1 : 0);  // sigmoid: the shared expert's gate row comes last
         // prompt-sized batches of a 16-bit engine: 128-row tiles on the tcgen05 grouped GEMM; otherwise 64-row tiles on mma.sync / SIMT
         const bool tc = !f32 && pairs >= 1024 && width % 8 == 0 && l.expert_ff % 8 == 0 && width >= 64 && l.expert_ff >= 64;
         const int tile = tc ? 128 : kMoeTileM;
@@ -1571,13 +1662,14 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
         // (a decode batch is a single 64-row tile there -- one CTA walking all of K -- so few tokens take the fp32 kernel as well)
         rc = NT >= 64 ? launch_dense_f32out(dt, h2, l.w_router, m->f32a, NT, outputs, width, st) : B200_ERR_UNSUPPORTED;
         if (rc == B200_ERR_UNSUPPORTED)
-            rc = dyt ? launch_proj_f32(dt, m->h, width, dt, l.w_router, nullptr, m->f32a, outputs, NT, outputs, width, st)
+            rc = dyt || sum_norm ? launch_proj_f32(dt, m->h, width, dt, l.w_router, nullptr, m->f32a, outputs, NT, outputs, width, st)
                      : launch_proj_f32(B200_F32, m->x, width, dt, l.w_router, nullptr, m->f32a, outputs, NT, outputs, width, st);
         if (rc != B200_OK) return rc;
         if (softmax) RUN(launch_moe_route_softmax(m->f32a, outputs, l.route_bias, sel_expert, sel_weight, NT, outputs, l.top, st));
-        else RUN(launch_moe_route_sigmoid(m->f32a, l.experts + 1, sel_expert, sel_weight, shared_gate, NT, l.experts, l.top, st));
+        else RUN(launch_moe_route_sigmoid(m->f32a, outputs, sel_expert, sel_weight, l.shared_ff > 0 ? shared_gate : nullptr, NT, l.experts, l.top, st));
         RUN(launch_moe_plan(sel_expert, sel_weight, row_token, row_weight, tile_expert, pair_row, n_live, NT, l.experts, l.top, tile, st));
-        if (softmax) RUN(launch_moe_gather_rows(dt, h2, row_token, m->xg, n_live, max_rows, width, tile, st));
+        if (softmax || sum_norm)  // sigmoid scores weigh the experts' inputs: the fp32 residual row, or the convolved row the router read
+            RUN(launch_moe_gather_rows(dt, h2, row_token, m->xg, n_live, max_rows, width, tile, st, softmax ? nullptr : row_weight));
         else RUN(launch_moe_gather(dt, m->x, row_token, row_weight, m->xg, n_live, max_rows, width, tile, st));
         const int n_up = inner_cols * l.expert_ff;
         const int up_act = l.gated ? -1 : l.act;
@@ -1586,7 +1678,7 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
         else RUN(launch_moe_grouped_gemm(dt, m->xg, l.w_up, m->u, tile_expert, n_live, max_tiles, n_up, width, up_act, st));
         if (l.gated) {
             inner += (size_t)max_rows * n_up * es;
-            RUN(launch_gated_activation(dt, m->u, inner, max_rows, l.expert_ff, l.act, n_live, tile, st));
+            RUN(launch_gated_activation(dt, m->u, inner, max_rows, l.expert_ff, l.act, n_live, tile, st, l.act_limit, l.act_slope));
         }
         if (tc) RUN(launch_gemm_tc_grouped(inner, l.w_down, m->yrows, max_rows, width, l.expert_ff, l.experts, tile_expert, n_live, -1, dt, st));
         else RUN(launch_moe_grouped_gemm(dt, inner, l.w_down, m->yrows, tile_expert, n_live, max_tiles, width, l.expert_ff, -1, st));
@@ -1595,14 +1687,16 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
             RUN(linear(m, h2, l.w_shared_up, m->us, NT, width, inner_cols * l.shared_ff, st));
             if (l.gated) {
                 sin += (size_t)NT * 2 * l.shared_ff * es;
-                RUN(launch_gated_activation(dt, m->us, sin, NT, l.shared_ff, l.act, nullptr, 0, st));
+                RUN(launch_gated_activation(dt, m->us, sin, NT, l.shared_ff, l.act, nullptr, 0, st, l.act_limit, l.act_slope));
             } else {
                 RUN(launch_activation(dt, m->us, (size_t)NT * l.shared_ff, l.act, st));
             }
             RUN(linear(m, sin, l.w_shared_down, m->ys, NT, l.shared_ff, width, st));
         }
         const void *y_shared = l.shared_ff > 0 ? m->ys : nullptr;
-        if (!softmax) {
+        if (sum_norm) {
+            RUN(sum_step(li, 1, nullptr, m->yrows, pair_row, y_shared, shared_gate, trace));
+        } else if (!softmax) {
             RUN(postnorm(nullptr, m->yrows, pair_row, l.top, y_shared, shared_gate, l.norm2, trace));
             h_normed = false;
         } else {

@@ -18,9 +18,10 @@ int launch_chunked_attention_tiles(int dtype, const void *q, const void *k_pool,
                                    int kv_heads, int dim, float scale, int chunk, cudaStream_t st);
 
 // attention_latent.cu (layouts in the file's header): proj [tokens, ld] holds q at column q_col and, when kv_col >= 0, the down-projection
+// (in kv_proj [tokens, kv_ld] instead, if given)
 int launch_latent_prep(int dtype, const void *proj, int ld, int q_col, int kv_col, void *qn, void *qr, void *pool, const float *kv_norm,
                        float eps, const int *tok_seq, const int *tok_pos, const int *block_table, int mpps, int tokens, int t_pad, int heads,
-                       int dim, int rot_dim, int kv_rank, int rot_dims, float rot_base, cudaStream_t st);
+                       int dim, int rot_dim, int kv_rank, int rot_dims, float rot_base, cudaStream_t st, const void *kv_proj = nullptr, int kv_ld = 0);
 int launch_latent_attention(int dtype, const void *ql, const void *qr, const void *pool, const float *sink, void *ol, const int *tok_seq,
                             const int *tok_pos, const int *block_table, int mpps, int tokens, int t_pad, int heads, int kv_rank, int rot_dim,
                             float scale, int window, int max_keys, cudaStream_t st, const int *tok_list = nullptr);
@@ -31,8 +32,11 @@ bool latent_attention_tiles_supported(int dtype, int kv_rank, int rot_dim);
 int launch_latent_attention_tiles(int dtype, const void *ql, const void *qr, const void *pool, const float *sink, void *ol, const int *tiles,
                                   int n_tiles, const int *block_table, int mpps, int t_pad, int heads, int kv_rank, int rot_dim, float scale,
                                   int window, int by_head, float *part, int part_tiles, cudaStream_t st);
+// head_gate: gate_in holds ONE number per head instead of one per value channel
 int launch_latent_gate(int dtype, const void *ov, const void *gate_in, int gate_ld, void *out, int tokens, int t_pad, int heads, int vdim,
-                       cudaStream_t st);
+                       cudaStream_t st, int head_gate = 0);
+// out [tokens, cols] = rmsnorm(in [tokens, ld] from its column 0 on) * w
+int launch_rms_rows(int dtype, const void *in, int ld, const float *w, float eps, void *out, int tokens, int cols, cudaStream_t st);
 
 // attention_scored.cu: proj [tokens, ld] holds q (heads*dim), k (kv_heads*dim), v (kv_heads*vdim) from column col0 on; b_in (optional) is
 // counted from the same row.  q_out [tokens, heads*dim]; pools K [pages, kv_heads, page, dim], V [pages, kv_heads, page, vdim]
@@ -100,6 +104,27 @@ int launch_decay_recurrent(const float *rec, float *S, float *o, const int *seq_
 int launch_group_output(int dtype, const float *o, const float *skip, int skip_ld, const float *w, float eps, const void *gate, int gate_ld,
                         int gate_act, int gate_first, void *out, int out_ld, int tokens, int cols, int groups, cudaStream_t st);
 
+// sum_norm.cu (the mechanisms' equations in the file's header)
+// one sublayer's input convolution: ring fp32 [slots, taps - 1, width], w fp32 [taps, width]; taps 0: none
+struct RingConv { float *ring = nullptr; const float *w = nullptr; int taps = 0; };
+// device arrays of the batch description: sequence and position of every packed row; first row, first position and slot of every portion
+struct PortionMap { const int *tok_seq, *tok_pos, *seq_start, *seq_pos0, *seq_slot; };
+// one_token: the host knows that every portion is a single token: h_out then receives the next sublayer's convolved input; otherwise
+// launch_conv_input forms it (next.taps == 0: h_out is the row itself either way)
+int launch_sum_norm(int dtype, float *x, const void *y_dense, const void *y_rows, const int *pair_row, int top, const void *y_shared,
+                    const float *shared_gate, float alpha, const float *g, float eps, int width, float *trace, void *h_out, RingConv own, RingConv next,
+                    int one_token, PortionMap pm, int tokens, cudaStream_t st);
+int launch_embed_pos(int dtype, const int *ids, const void *table, float *x, void *h_out, int width, int vocab, float scale, float base, RingConv next,
+                     int one_token, PortionMap pm, int tokens, cudaStream_t st);
+int launch_conv_input(int dtype, const float *x, void *h, int width, RingConv cv, PortionMap pm, int tokens, cudaStream_t st);
+
+// mingru.cu: proj row z | u | gate (cols each), bias [2 * cols] or NULL, state fp32 [slots, cols]; out [tokens, cols].  Portions of at least
+// kMingruShort tokens arrive as chunks, int4 {sequence, first packed row, tokens, index in its portion}, a portion's chunks in order; maps: fp32
+// scratch [n_chunks, 2, cols].  n_short: tokens in shorter portions (0: their kernel is not launched)
+constexpr int kMingruShort = 8;
+int launch_mingru(int dtype, const void *proj, int ld, const float *bias, float *state, float *maps, void *out, const int *chunks, int n_chunks,
+                  const int *seq_start, const int *seq_pos0, const int *seq_slot, int n_seqs, int n_short, int cols, cudaStream_t st);
+
 // gla.cu
 // decay[t, c] = sigmoid(z)^(1/tau), z = w_decay[c, :] . proj[t, col0 : col0 + rank] + bias[c]   (fp32 from the projection on)
 int launch_gla_decay(int dtype, const void *proj, int ld, int col0, const void *w_decay, const float *bias, float tau, float *decay,
@@ -128,11 +153,15 @@ int launch_moe_plan(const int *sel_expert, const float *sel_weight, int *row_tok
 // xg[row, :] = T(weight[row] * x[token[row], :]) (zeros for padding rows): the routing weight multiplies the expert's INPUT
 int launch_moe_gather(int dtype, const float *x, const int *row_token, const float *row_weight, void *xg, const int *n_tiles,
                       int max_rows, int width, int tile, cudaStream_t st);
-// xg[row, :] = h[token[row], :] of the engine dtype (zeros for padding rows)
+// xg[row, :] = h[token[row], :] of the engine dtype (zeros for padding rows), times row_weight[row] if given
 int launch_moe_gather_rows(int dtype, const void *h, const int *row_token, void *xg, const int *n_tiles, int max_rows, int width, int tile,
-                           cudaStream_t st);
+                           cudaStream_t st, const float *row_weight = nullptr);
 // out[r, c] = act(in[r, c]) * in[r, inner + c], in [rows, 2 * inner]; n_tiles (optional, device): only rows < *n_tiles * tile are live
-int launch_gated_activation(int dtype, const void *in, void *out, int rows, int inner, int act, const int *n_tiles, int tile, cudaStream_t st);
+// limit, slope: parameters of B200_ACT_CLAMP_GLU
+int launch_gated_activation(int dtype, const void *in, void *out, int rows, int inner, int act, const int *n_tiles, int tile, cudaStream_t st,
+                            float limit = 0.0f, float slope = 0.0f);
+// in place, row by row: x = a n(x) + b n(x^2) + c n(x^3) + e with coef [4] = a, b, c, e, n(v) = v / sqrt(mean over the row of v^2 + eps)
+int launch_poly_norm(int dtype, void *x, const float *coef, float eps, int rows, int cols, cudaStream_t st);
 // in place: x[r, c] = act(x[r, c] + bias[c]); bias NULL: none; act < 0: none
 int launch_bias_activation(int dtype, void *x, const float *bias, size_t rows, int cols, int act, cudaStream_t st);
 // gemm_tc.cu: the same product on tcgen05 for row tiles of 128 (16-bit dtypes, K >= 64 and a multiple of 8; B200_ERR_UNSUPPORTED otherwise)

@@ -155,15 +155,36 @@ moe_gather_kernel(const float *__restrict__ x, const int *__restrict__ row_token
         xg[(size_t)r * width + c] = Elem<T>::from_f(t >= 0 ? w * x[(size_t)t * width + c] : 0.0f);
 }
 
-// xg[row, :] = h[token[row], :] (zeros for padding rows): the expert reads the token's row as it is, the weight goes on its output
+// xg[row, :] = h[token[row], :] (zeros for padding rows): the expert reads the token's row as it is and the weight goes on its output, or
+// (row_weight given) the row times its weight, for a weight on the input of experts that read a row of the engine dtype
 template <typename T>
 __global__ void __launch_bounds__(128)
 moe_gather_rows_kernel(const T *__restrict__ h, const int *__restrict__ row_token, T *__restrict__ xg, const int *__restrict__ n_tiles, int width,
-                       int tile) {
+                       int tile, const float *__restrict__ row_weight) {
     const int r = blockIdx.x;
     if (r >= *n_tiles * tile) return;
     const int t = row_token[r];
     constexpr int V = Elem<T>::kVec;
+    if (row_weight) {
+        const float w = row_weight[r];
+        if (width % V == 0 && ((reinterpret_cast<size_t>(h) | reinterpret_cast<size_t>(xg)) & 15) == 0) {
+            for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+                uint4 piece = make_uint4(0, 0, 0, 0);
+                if (t >= 0) {
+                    float f[V];
+                    unpack16<T>(ld_v4(h + (size_t)t * width + c), f);
+#pragma unroll
+                    for (int e = 0; e < V; ++e) f[e] *= w;
+                    piece = pack16<T>(f);
+                }
+                st_v4(xg + (size_t)r * width + c, piece);
+            }
+            return;
+        }
+        for (int c = threadIdx.x; c < width; c += blockDim.x)
+            xg[(size_t)r * width + c] = Elem<T>::from_f(t >= 0 ? w * Elem<T>::to_f(h[(size_t)t * width + c]) : 0.0f);
+        return;
+    }
     if (width % V == 0 && ((reinterpret_cast<size_t>(h) | reinterpret_cast<size_t>(xg)) & 15) == 0) {
         for (int c = threadIdx.x * V; c < width; c += blockDim.x * V)
             st_v4(xg + (size_t)r * width + c, t >= 0 ? ld_v4(h + (size_t)t * width + c) : make_uint4(0, 0, 0, 0));
@@ -172,11 +193,20 @@ moe_gather_rows_kernel(const T *__restrict__ h, const int *__restrict__ row_toke
     for (int c = threadIdx.x; c < width; c += blockDim.x) xg[(size_t)r * width + c] = t >= 0 ? h[(size_t)t * width + c] : Elem<T>::from_f(0.0f);
 }
 
+// g = min(gate, limit), u = clamp(up, -limit, limit): g * sigmoid(slope * g) * (u + 1); limit <= 0: no clamp
+__device__ __forceinline__ float gated_apply(float g, float u, int act, float limit, float slope) {
+    if (act == B200_ACT_CLAMP_GLU) {
+        if (limit > 0.0f) g = fminf(g, limit), u = fminf(fmaxf(u, -limit), limit);
+        return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
+    }
+    return act_apply(g, act) * u;
+}
+
 // out[r, c] = act(in[r, c]) * in[r, inner + c] for rows r < *n_tiles * tile (all `rows` when n_tiles is NULL); in [rows, 2 * inner].
 // One 16-byte piece of the output per thread when the rows start on 16-byte boundaries, else one element.
 template <typename T>
 __global__ void gated_activation_kernel(const T *__restrict__ in, T *__restrict__ out, int rows, int inner, int act, const int *__restrict__ n_tiles,
-                                        int tile) {
+                                        int tile, float limit, float slope) {
     constexpr int V = Elem<T>::kVec;
     const int live = n_tiles ? min(rows, *n_tiles * tile) : rows;
     if (inner % V == 0 && ((reinterpret_cast<size_t>(in) | reinterpret_cast<size_t>(out)) & 15) == 0) {
@@ -188,7 +218,7 @@ __global__ void gated_activation_kernel(const T *__restrict__ in, T *__restrict_
             unpack16<T>(ld_v4(in + r * 2 * inner + c), g);
             unpack16<T>(ld_v4(in + r * 2 * inner + inner + c), u);
 #pragma unroll
-            for (int e = 0; e < V; ++e) g[e] = act_apply(g[e], act) * u[e];
+            for (int e = 0; e < V; ++e) g[e] = gated_apply(g[e], u[e], act, limit, slope);
             st_v4(out + r * inner + c, pack16<T>(g));
         }
         return;
@@ -197,7 +227,7 @@ __global__ void gated_activation_kernel(const T *__restrict__ in, T *__restrict_
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
         const size_t r = i / inner, c = i - r * inner;
         const float g = Elem<T>::to_f(in[r * 2 * inner + c]), u = Elem<T>::to_f(in[r * 2 * inner + inner + c]);
-        out[i] = Elem<T>::from_f(act_apply(g, act) * u);
+        out[i] = Elem<T>::from_f(gated_apply(g, u, act, limit, slope));
     }
 }
 
@@ -231,6 +261,68 @@ __global__ void bias_activation_kernel(T *__restrict__ x, const float *__restric
         float v = Elem<T>::to_f(x[i]);
         if (bias) v += bias[i % cols];
         x[i] = Elem<T>::from_f(act >= 0 ? act_apply(v, act) : v);
+    }
+}
+
+// In place, one CTA per row: x = a n(x) + b n(x^2) + c n(x^3) + e, n(v) = v / sqrt(mean over the row of v^2 + eps).  One pass forms the three
+// mean squares (of x, x^2 and x^3) together; a thread's pieces stay in registers in between when the row is short enough.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(512)
+poly_norm_kernel(T *__restrict__ x, const float *__restrict__ coef, float eps, int cols) {
+    constexpr int N = VEC ? Elem<T>::kVec : 1, KP = VEC ? 2 : 8;
+    __shared__ float red[3][17];
+    T *row = x + (size_t)blockIdx.x * cols;
+    auto load = [&](int c, float *v) {
+        if constexpr (VEC) unpack16<T>(ld_v4(row + c), v);
+        else v[0] = Elem<T>::to_f(row[c]);
+    };
+    float s1 = 0.0f, s2 = 0.0f, s3 = 0.0f;
+    auto add = [&](const float *v) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const float q = v[i] * v[i];
+            s1 += q, s2 = fmaf(q, q, s2), s3 = fmaf(q * q, q, s3);
+        }
+    };
+    const bool held = cols <= (int)blockDim.x * N * KP;
+    float keep[KP][N];
+    if (held) {
+#pragma unroll
+        for (int i = 0; i < KP; ++i) {
+            const int c = (threadIdx.x + i * blockDim.x) * N;
+            if (c < cols) load(c, keep[i]), add(keep[i]);
+        }
+    } else {
+        for (int c = threadIdx.x * N; c < cols; c += blockDim.x * N) {
+            float v[N];
+            load(c, v), add(v);
+        }
+    }
+    s1 = warp_sum(s1), s2 = warp_sum(s2), s3 = warp_sum(s3);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
+    if (lane == 0) red[0][warp] = s1, red[1][warp] = s2, red[2][warp] = s3;
+    __syncthreads();
+    s1 = s2 = s3 = 0.0f;
+    for (int w = 0; w < nwarp; ++w) s1 += red[0][w], s2 += red[1][w], s3 += red[2][w];
+    const float n = (float)cols;
+    const float a = coef[0] * rsqrtf(s1 / n + eps), b = coef[1] * rsqrtf(s2 / n + eps), d = coef[2] * rsqrtf(s3 / n + eps), e0 = coef[3];
+    auto finish = [&](int c, float *v) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = fmaf(v[i], fmaf(v[i], fmaf(v[i], d, b), a), e0);
+        if constexpr (VEC) st_v4(row + c, pack16<T>(v));
+        else row[c] = Elem<T>::from_f(v[0]);
+    };
+    if (held) {
+#pragma unroll
+        for (int i = 0; i < KP; ++i) {
+            const int c = (threadIdx.x + i * blockDim.x) * N;
+            if (c < cols) finish(c, keep[i]);
+        }
+        return;
+    }
+    for (int c = threadIdx.x * N; c < cols; c += blockDim.x * N) {
+        float v[N];
+        load(c, v), finish(c, v);
     }
 }
 
@@ -424,17 +516,18 @@ int launch_moe_route_softmax(const float *logits, int ld, const float *bias, int
 }
 
 int launch_moe_gather_rows(int dtype, const void *h, const int *row_token, void *xg, const int *n_tiles, int max_rows, int width, int tile,
-                           cudaStream_t st) {
+                           cudaStream_t st, const float *row_weight) {
     if (max_rows == 0) return B200_OK;
-    B200_DISPATCH_DTYPE(dtype, { moe_gather_rows_kernel<T><<<max_rows, 128, 0, st>>>((const T *)h, row_token, (T *)xg, n_tiles, width, tile); });
+    B200_DISPATCH_DTYPE(dtype, { moe_gather_rows_kernel<T><<<max_rows, 128, 0, st>>>((const T *)h, row_token, (T *)xg, n_tiles, width, tile, row_weight); });
     return cuda_status("moe_gather_rows launch");
 }
 
-int launch_gated_activation(int dtype, const void *in, void *out, int rows, int inner, int act, const int *n_tiles, int tile, cudaStream_t st) {
+int launch_gated_activation(int dtype, const void *in, void *out, int rows, int inner, int act, const int *n_tiles, int tile, cudaStream_t st,
+                            float limit, float slope) {
     if (rows == 0 || inner == 0) return B200_OK;
     const size_t n = (size_t)rows * inner / 4;
     const unsigned grid = (unsigned)std::max<size_t>(1, std::min<size_t>((n + 255) / 256, 148 * 16));
-    B200_DISPATCH_DTYPE(dtype, { gated_activation_kernel<T><<<grid, 256, 0, st>>>((const T *)in, (T *)out, rows, inner, act, n_tiles, tile); });
+    B200_DISPATCH_DTYPE(dtype, { gated_activation_kernel<T><<<grid, 256, 0, st>>>((const T *)in, (T *)out, rows, inner, act, n_tiles, tile, limit, slope); });
     return cuda_status("gated_activation launch");
 }
 
@@ -444,6 +537,18 @@ int launch_bias_activation(int dtype, void *x, const float *bias, size_t rows, i
     const unsigned grid = (unsigned)std::max<size_t>(1, std::min<size_t>((n + 255) / 256, 148 * 16));
     B200_DISPATCH_DTYPE(dtype, { bias_activation_kernel<T><<<grid, 256, 0, st>>>((T *)x, bias, rows, cols, act); });
     return cuda_status("bias_activation launch");
+}
+
+int launch_poly_norm(int dtype, void *x, const float *coef, float eps, int rows, int cols, cudaStream_t st) {
+    if (rows == 0 || cols == 0) return B200_OK;
+    B200_DISPATCH_DTYPE(dtype, {
+        const bool vec = cols % Elem<T>::kVec == 0 && (reinterpret_cast<size_t>(x) & 15) == 0;
+        const int per = vec ? Elem<T>::kVec : 1;
+        const int threads = std::min(512, std::max(32, ((cols + per - 1) / per + 31) / 32 * 32));
+        auto kern = vec ? poly_norm_kernel<T, true> : poly_norm_kernel<T, false>;
+        kern<<<rows, threads, 0, st>>>((T *)x, coef, eps, cols);
+    });
+    return cuda_status("poly_norm launch");
 }
 
 int launch_moe_plan(const int *sel_expert, const float *sel_weight, int *row_token, float *row_weight, int *tile_expert, int *pair_row,
@@ -510,4 +615,10 @@ extern "C" int b200_moe_route_softmax(const float *logits, int ld, const float *
     B200_REQUIRE(logits && sel_expert && sel_weight, "moe_route_softmax: null pointer");
     B200_REQUIRE(tokens >= 0 && outputs > 0 && top > 0 && top <= outputs && ld >= outputs, "moe_route_softmax: bad shape");
     return launch_moe_route_softmax(logits, ld, bias, sel_expert, sel_weight, tokens, outputs, top, as_stream(stream));
+}
+
+extern "C" int b200_poly_norm(void *x, const float *coef, float eps, int rows, int cols, int dtype, b200_stream_t stream) {
+    B200_REQUIRE(x && coef, "poly_norm: null pointer");
+    B200_REQUIRE(rows >= 0 && cols >= 0, "poly_norm: bad shape");
+    return launch_poly_norm(dtype, x, coef, eps, rows, cols, as_stream(stream));
 }

@@ -74,9 +74,9 @@ def fuse_layer(spec, get, width, dtype, device):
     spec["norm1"] = vec("norm1")
     if spec["mlp"] == m.MLP_MOE:
         E = spec["experts"]
-        gate_row = get("mlp.shared.sg").reshape(1, width) if spec["shared_ff"] else torch.zeros(1, width)
+        router = [get("mlp.router").float()] + ([get("mlp.shared.sg").reshape(1, width).float()] if spec["shared_ff"] else [])
         spec.update(norm2=vec("norm2"),
-                    w_router=torch.cat([get("mlp.router").float(), gate_row.float()], 0).to(device=device, dtype=dtype).contiguous(),
+                    w_router=torch.cat(router, 0).to(device=device, dtype=dtype).contiguous(),
                     w_up=torch.stack([get(f"mlp.e{e}.up") for e in range(E)]).to(device=device, dtype=dtype).contiguous(),
                     w_down=torch.stack([get(f"mlp.e{e}.down") for e in range(E)]).to(device=device, dtype=dtype).contiguous())
         if spec["shared_ff"]:
