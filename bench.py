@@ -1143,46 +1143,46 @@ LATENT_SIZES = {  # Zefenex-shaped layer lists: four latent-attention layers, th
 }
 
 
-def run_latent(args):
-    """--mode latent: prefill and decode throughput of a Zefenex-shaped model (random weights, bf16) on the layer-list decoder at one of
-    LATENT_SIZES and, in the same process, of the framework's closest other design at equal size: a Vasolix-shaped model of four chunked-
-    attention layers with the same width, head count, window (as its chunk) and expert sizes.  Prefill: one prompt of --prefill-tokens tokens
-    in one engine call.  Decode: --batch sequences with --ctx cached positions each, one token per sequence per step, through the call a
-    served request takes (host batch description in, device logits out)."""
-    import numpy as np
-    import torch
+class LayerListBench:
+    """What the latent-attention measurements share: random tensors, CUDA-event timing with clock samples, prefill and decode of one engine
+    through HybridDecoder.forward."""
 
-    mod = importlib.import_module("llm-inference-engine_b200")
-    mod.lib()
-    sz = LATENT_SIZES[args.latent_size]
-    W, H, M, V = sz["width"], sz["heads"], sz["moe"], 32000
-    dev = torch.device("cuda", 0)
-    torch.cuda.set_device(dev)
-    gen = torch.Generator().manual_seed(7)
+    def __init__(self, args, mod, ctx):
+        import torch
 
-    def rnd(*shape, std=0.02):
-        return (torch.randn(*shape, generator=gen) * std).to(torch.bfloat16)
+        self.args, self.ctx, self.vocab = args, ctx, 32000
+        self.dev = torch.device("cuda", 0)
+        torch.cuda.set_device(self.dev)
+        self.gen = torch.Generator().manual_seed(7)
+        self.tokens, self.batch = args.prefill_tokens, args.batch
+        page = mod.KV_PAGE_SIZE
+        self.per_seq = (max(self.tokens, ctx + args.steps + args.warmup + 8) + page - 1) // page
+        self.limits = dict(dtype="bfloat16", device=self.dev, max_tokens=max(self.tokens, self.batch, 2048), max_seqs=max(self.batch, 1), max_pages_per_seq=self.per_seq)
+        self.ids = torch.randint(0, self.vocab, (max(self.tokens, ctx + 1),), generator=self.gen).tolist()
+        self.peaks = {}
+        try:
+            self.peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
+        except Exception:
+            pass
 
-    def ones(n):
+    def rnd(self, *shape, std=0.02):
+        import torch
+
+        return (torch.randn(*shape, generator=self.gen) * std).to(torch.bfloat16)
+
+    def ones(self, n):
+        import torch
+
         return torch.ones(n, dtype=torch.bfloat16)
 
-    Tq, B, ctx = args.prefill_tokens, args.batch, args.ctx
-    if ctx % sz["window"] == 0:
-        ctx += sz["window"] // 2  # a context that ends exactly on a chunk edge would leave the chunked model's decoded token a single key to look at
-    page = mod.KV_PAGE_SIZE
-    per_seq = (max(Tq, ctx + args.steps + args.warmup + 8) + page - 1) // page
-    peaks = {}
-    try:
-        peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
-    except Exception:
-        pass
+    def timed(self, fn, steps, warmup):
+        import torch
 
-    def timed(fn, steps, warmup):
         for _ in range(warmup):
             fn()
         torch.cuda.synchronize()
         e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        with ClockSampler(0, gpu_uuid(dev)) as clocks:
+        with ClockSampler(0, gpu_uuid(self.dev)) as clocks:
             e0.record()
             for _ in range(steps):
                 fn()
@@ -1190,10 +1190,13 @@ def run_latent(args):
             torch.cuda.synchronize()
         return e0.elapsed_time(e1) / steps, clocks.summary()
 
-    def measure(eng, ids, flops_prefill, bytes_decode):
+    def measure(self, eng, flops_prefill, bytes_decode):
+        import numpy as np
+
+        args, ids, Tq, B, per_seq, ctx = self.args, self.ids, self.tokens, self.batch, self.per_seq, self.ctx
         eng.set_pools(per_seq * max(B, 1), max(B, 1))
         bt = np.arange(per_seq * max(B, 1), dtype=np.int32).reshape(max(B, 1), per_seq)
-        pre_ms, pre_clocks = timed(lambda: eng.forward(ids[:Tq], [0, Tq], [0], [0], bt[:1].reshape(-1), [Tq - 1]), max(3, min(args.steps, 20)), 3)
+        pre_ms, pre_clocks = self.timed(lambda: eng.forward(ids[:Tq], [0, Tq], [0], [0], bt[:1].reshape(-1), [Tq - 1]), max(3, min(args.steps, 20)), 3)
         for b in range(B):
             eng.forward(ids[:ctx], [0, ctx], [0], [b], bt[b:b + 1].reshape(-1), [])
         state = {"pos": ctx}
@@ -1202,24 +1205,32 @@ def run_latent(args):
             eng.forward(ids[:B], list(range(B + 1)), [state["pos"]] * B, list(range(B)), bt.reshape(-1), list(range(B)))
             state["pos"] += 1
 
-        dec_ms, dec_clocks = timed(step, args.steps, max(args.warmup, 3))
+        dec_ms, dec_clocks = self.timed(step, args.steps, max(args.warmup, 3))
         pre_tflops = flops_prefill / (pre_ms * 1e-3) / 1e12
         dec_gbs = bytes_decode / (dec_ms * 1e-3) / 1e9
         return {"prefill": {"tokens_per_s": Tq * 1e3 / pre_ms, "ms": pre_ms, "tflops": pre_tflops,
-                            "frac_of_measured_bf16_sustained": pre_tflops / float(peaks.get("bf16_tflops_sustained", 1400.0)), "clocks": pre_clocks},
+                            "frac_of_measured_bf16_sustained": pre_tflops / float(self.peaks.get("bf16_tflops_sustained", 1400.0)), "clocks": pre_clocks},
                 "decode": {"tokens_per_s": B * 1e3 / dec_ms, "ms_per_step": dec_ms, "algorithmic_gb_per_s": dec_gbs,
-                           "frac_of_measured_hbm": dec_gbs / float(peaks.get("hbm_gbs", 6650.0)), "clocks": dec_clocks}}
+                           "frac_of_measured_hbm": dec_gbs / float(self.peaks.get("hbm_gbs", 6650.0)), "clocks": dec_clocks}}
 
-    ids = torch.randint(0, V, (max(Tq, ctx + 1),), generator=gen).tolist()
+
+def zefenex_model(lb, sz):
+    """The Zefenex-shaped model of the numbers `sz` (window 0: plain causal; identity / shared 0: none), with the FLOPs of its prefill and the
+    bytes of its decode step."""
+    import torch
+
+    W, H, M, V, Tq, B, window = sz["width"], sz["heads"], sz["moe"], lb.vocab, lb.tokens, lb.batch, sz["window"]
+    rnd, ones = lb.rnd, lb.ones
     touched = min(M["experts"], B * M["top"])
-    window = sz["window"]
-    keys_of = lambda pos: min(pos + 1, window)
+    keys_of = lambda pos: min(pos + 1, window) if window else pos + 1
     pair_sum = float(sum(keys_of(i) for i in range(Tq)))
-
-    # ---- the Zefenex-shaped model
     d, dr, dv, r = sz["dim"], sz["rot"], sz["vdim"], sz["rank"]
-    mixer = {"heads": H, "dim": d, "rot_dim": dr, "vdim": dv, "kv_rank": r, "scale": (d + dr) ** -0.5, "mask": {"size": window}, "rot": {"base": 10000.0, "dims": dr}}
-    moe = {"kind": "moe", "expert": {"ff": M["ff"]}, "router": {"experts": M["experts"], "identity": M["identity"], "top": M["top"]}, "shared": {"ff": M["shared"]}}
+    mixer = {"heads": H, "dim": d, "rot_dim": dr, "vdim": dv, "kv_rank": r, "scale": (d + dr) ** -0.5, "rot": {"base": 10000.0, "dims": dr}}
+    if window:
+        mixer["mask"] = {"size": window}
+    moe = {"kind": "moe", "expert": {"ff": M["ff"]}, "router": {"experts": M["experts"], "identity": M["identity"], "top": M["top"]}}
+    if M["shared"]:
+        moe["shared"] = {"ff": M["shared"]}
     layers = [{"type": "latent_attention", "mixer": dict(mixer), "mlp": {"kind": "dense", "ff": sz["dense_ff"]}},
               {"type": "latent_attention", "mixer": dict(mixer, kv_from=0), "mlp": moe},
               {"type": "latent_attention", "mixer": dict(mixer), "mlp": moe},
@@ -1253,17 +1264,44 @@ def run_latent(args):
             gate, up, down = rnd(M["experts"], M["ff"], W), rnd(M["experts"], M["ff"], W), rnd(M["experts"], W, M["ff"])
             for e in range(M["experts"]):
                 t[f"{p}mlp.e{e}.gate"], t[f"{p}mlp.e{e}.up"], t[f"{p}mlp.e{e}.down"] = gate[e], up[e], down[e]
-            t.update({p + "mlp.shared.gate": rnd(M["shared"], W), p + "mlp.shared.up": rnd(M["shared"], W), p + "mlp.shared.down": rnd(W, M["shared"])})
+            if M["shared"]:
+                t.update({p + "mlp.shared.gate": rnd(M["shared"], W), p + "mlp.shared.up": rnd(M["shared"], W), p + "mlp.shared.down": rnd(W, M["shared"])})
             lat_moe_params += 1
     zef = importlib.import_module("llm-inference-engine_b200.models.zefenex")
-    model = zef.ZefenexModel(config, t, dtype="bfloat16", device=dev, max_tokens=max(Tq, B, 2048), max_seqs=max(B, 1), max_pages_per_seq=per_seq)
+    model = zef.ZefenexModel(config, t, **lb.limits)
     moe_active = 3 * W * (M["top"] * M["ff"] + M["shared"]) + W * (M["experts"] + M["identity"])
     lat_active = lat_params + lat_dense_params + lat_moe_params * moe_active
     lat_attn_flops = 2.0 * len(layers) * H * ((r + dr) + r) * pair_sum
     lat_w_bytes = 2 * (lat_params + lat_dense_params + lat_moe_params * (3 * W * (touched * M["ff"] + M["shared"]) + W * (M["experts"] + M["identity"]))) + 2 * V * W
-    lat_kv_bytes = 2.0 * len(layers) * B * (r + dr) * keys_of(ctx)   # every layer reads the window's rows once (the heads share them)
-    latent = measure(model.engine, ids, 2.0 * Tq * lat_active + lat_attn_flops, lat_w_bytes + lat_kv_bytes)
-    del model, t
+    lat_kv_bytes = 2.0 * len(layers) * B * (r + dr) * keys_of(lb.ctx)   # every layer reads the window's rows once (the heads share them)
+    return model, 2.0 * lb.tokens * lat_active + lat_attn_flops, lat_w_bytes + lat_kv_bytes
+
+
+def run_latent(args):
+    """--mode latent: prefill and decode throughput of a Zefenex-shaped model (random weights, bf16) on the layer-list decoder at one of
+    LATENT_SIZES and, in the same process, of the framework's closest other design at equal size: a Vasolix-shaped model of four chunked-
+    attention layers with the same width, head count, window (as its chunk) and expert sizes.  Prefill: one prompt of --prefill-tokens tokens
+    in one engine call.  Decode: --batch sequences with --ctx cached positions each, one token per sequence per step, through the call a
+    served request takes (host batch description in, device logits out)."""
+    import torch
+
+    mod = importlib.import_module("llm-inference-engine_b200")
+    mod.lib()
+    sz = LATENT_SIZES[args.latent_size]
+    W, H, M, V = sz["width"], sz["heads"], sz["moe"], 32000
+    d, dr, r = sz["dim"], sz["rot"], sz["rank"]
+    Tq, B, ctx = args.prefill_tokens, args.batch, args.ctx
+    if ctx % sz["window"] == 0:
+        ctx += sz["window"] // 2  # a context that ends exactly on a chunk edge would leave the chunked model's decoded token a single key to look at
+    lb = LayerListBench(args, mod, ctx)
+    rnd, ones = lb.rnd, lb.ones
+    touched = min(M["experts"], B * M["top"])
+    window = sz["window"]
+
+    # ---- the Zefenex-shaped model
+    model, flops, n_bytes = zefenex_model(lb, sz)
+    latent = lb.measure(model.engine, flops, n_bytes)
+    del model
     torch.cuda.empty_cache()
 
     # ---- the closest other design at equal size: four chunked-attention layers (values = keys, whole-projection norms), sigmoid-routed experts
@@ -1283,13 +1321,13 @@ def run_latent(args):
             t[f"{p}mlp.e{e}.up"], t[f"{p}mlp.e{e}.down"] = up[e], down[e]
         t.update({p + "mlp.shared.up": rnd(M["shared"], W), p + "mlp.shared.down": rnd(W, M["shared"]), p + "mlp.shared.sg": rnd(1, W)})
     vas = importlib.import_module("llm-inference-engine_b200.models.vasolix")
-    vmodel = vas.VasolixModel(vconfig, t, dtype="bfloat16", device=dev, max_tokens=max(Tq, B, 2048), max_seqs=max(B, 1), max_pages_per_seq=per_seq)
+    vmodel = vas.VasolixModel(vconfig, t, **lb.limits)
     v_att = W * (2 * H + Gk) * d + H * d * W
     v_moe = 2 * W * (M["top"] * M["ff"] + M["shared"]) + W * (M["experts"] + 1)
     chunk_pairs = float(sum(i % window + 1 for i in range(Tq)))
     v_flops = 2.0 * Tq * 4 * (v_att + v_moe) + 2.0 * 4 * 2 * H * d * chunk_pairs
     v_bytes = 2 * 4 * (v_att + 2 * W * (touched * M["ff"] + M["shared"]) + W * (M["experts"] + 1)) + 2 * V * W + 2.0 * 4 * 2 * B * Gk * d * (ctx % window + 1)
-    closest = measure(vmodel.engine, ids, v_flops, v_bytes)
+    closest = lb.measure(vmodel.engine, v_flops, v_bytes)
     print(json.dumps({
         "metric": "latent-attention model prefill / decode tokens/s", "value": latent["prefill"]["tokens_per_s"], "unit": "tokens/s (prefill)", "n_gpus": 1,
         "steps": args.steps, "warmup": max(args.warmup, 3), "higher_is_better": True, "dtype": "bf16", "data": "synthetic", "impl": "b200",
@@ -1298,6 +1336,91 @@ def run_latent(args):
                    "closest": f"Vasolix-shaped: width {W}, 4 chunked-attention layers ({H} heads over {Gk} kv heads, dim {d}, chunk {window}), {M['experts']} experts top {M['top']}",
                    "prefill_tokens": Tq, "decode_batch": B, "decode_context": ctx, "cache_policy": "weights larger than L2 at sizes m and l; no explicit flush"},
         "latent": latent, "closest": closest,
+        "e2e": "all numbers are taken through HybridDecoder.forward: host batch description in (one H2D copy per call), device logits out"}), flush=True)
+
+
+SUM_NORM_SIZES = {  # Zasapel-shaped layer lists (minGRU with a dense feed-forward, two latent layers of which the second reads the first's rows and
+    # a minGRU, with experts).  Widths, heads, ranks, dense and expert sizes follow LATENT_SIZES, so that the Zefenex-shaped model of the same
+    # numbers (without window, identity experts and shared expert, which this design does not have) stands beside it.
+    "s": dict(LATENT_SIZES["s"], rnn=1536, q_rank=384, taps=4),
+    "m": dict(LATENT_SIZES["m"], rnn=3072, q_rank=768, taps=4),
+    "l": dict(LATENT_SIZES["l"], rnn=6144, q_rank=1536, taps=4),
+}
+
+
+def zasapel_model(lb, sz):
+    """The Zasapel-shaped model of the numbers `sz`, with the FLOPs of its prefill and the bytes of its decode step."""
+    rnd, ones, Tq, B, V = lb.rnd, lb.ones, lb.tokens, lb.batch, lb.vocab
+    W, H, M, R, rq, d, dv, r = sz["width"], sz["heads"], sz["moe"], sz["rnn"], sz["q_rank"], sz["dim"], sz["vdim"], sz["rank"]
+    rnn = {"type": "mingru", "mixer": {"width": R}}
+    att = {"type": "latent_attention", "mixer": {"heads": H, "dim": d, "vdim": dv, "kv_rank": r, "q_rank": rq, "scale": d ** -0.5}}
+    moe = {"kind": "moe", "expert": {"ff": M["ff"], "limit": 7.0}, "router": {"experts": M["experts"], "top": M["top"]}}
+    layers = [dict(rnn, mlp={"kind": "dense", "ff": sz["dense_ff"]}), dict(att, mlp=moe),
+              dict(att, mixer=dict(att["mixer"], kv_from=1), mlp=moe), dict(rnn, mlp=moe)]
+    config = {"architecture": "Zasapel", "width": W, "vocab": V, "canon": {"taps": sz["taps"]}, "norm": {"eps": 1e-6}, "postln_alpha": 2.0, "layers": layers}
+    t = {"embed": rnd(V, W, std=1.0), "head": rnd(V, W), "final.norm": rnd(W)}
+    params = 0
+    for i, layer in enumerate(layers):
+        p = f"l{i}."
+        for k in ("1", "2"):
+            t[p + "norm" + k], t[p + "canon" + k] = rnd(W), rnd(W, sz["taps"], std=0.3)
+        if layer["type"] == "mingru":
+            t.update({p + "mix." + k: rnd(R, W) for k in ("z", "x", "g")})
+            t.update({p + "mix.z.b": rnd(R), p + "mix.x.b": rnd(R), p + "mix.o": rnd(W, R)})
+            params += 4 * W * R
+        else:
+            t.update({p + "mix.dq": rnd(rq, W), p + "mix.dq.norm": ones(rq), p + "mix.uq": rnd(H * d, rq), p + "mix.uk": rnd(H * d, r, std=0.05),
+                      p + "mix.uv": rnd(H * dv, r, std=0.05), p + "mix.g": rnd(H, W), p + "mix.o": rnd(W, H * dv)})
+            params += W * rq + rq * H * d + H * d * r + H * dv * r + H * W + W * H * dv
+            if "kv_from" not in layer["mixer"]:
+                t.update({p + "mix.dkv": rnd(r, W), p + "mix.dkv.norm": ones(r)})
+                params += W * r
+        if layer["mlp"]["kind"] == "dense":
+            t.update({p + "mlp.up": rnd(sz["dense_ff"], W), p + "mlp.down": rnd(W, sz["dense_ff"]), p + "mlp.act": rnd(4, std=0.5)})
+            params += 2 * W * sz["dense_ff"]
+        else:
+            t[p + "mlp.router"] = rnd(M["experts"], W)
+            gate, up, down = rnd(M["experts"], M["ff"], W), rnd(M["experts"], M["ff"], W), rnd(M["experts"], W, M["ff"])
+            for e in range(M["experts"]):
+                t[f"{p}mlp.e{e}.gate"], t[f"{p}mlp.e{e}.up"], t[f"{p}mlp.e{e}.down"] = gate[e], up[e], down[e]
+    model = importlib.import_module("llm-inference-engine_b200.models.zasapel").ZasapelModel(config, t, **lb.limits)
+    n_att, n_moe, n_rnn, touched = 2, 3, 2, min(M["experts"], B * M["top"])
+    moe_active = 3 * W * M["top"] * M["ff"] + W * M["experts"]
+    flops = 2.0 * Tq * (params + n_moe * moe_active) + 2.0 * n_att * H * 2 * r * (Tq * (Tq + 1) / 2.0)
+    n_bytes = 2 * (params + n_moe * (3 * W * touched * M["ff"] + W * M["experts"]) + V * W) + 2.0 * n_att * B * r * (lb.ctx + 1) + 8.0 * n_rnn * B * R + \
+        2 * len(layers) * B * sz["taps"] * 4.0 * W
+    return model, flops, n_bytes
+
+
+def run_zasapel(args):
+    """--mode zasapel: prefill and decode throughput of a Zasapel-shaped model (random weights, bf16) on the layer-list decoder at one of
+    SUM_NORM_SIZES and, in the same process, of the framework's closest other design at equal size: the Zefenex-shaped model (latent
+    attention, dense and routed gated feed-forwards).  Prefill: one prompt of --prefill-tokens tokens in one engine call.  Decode: --batch
+    sequences with --ctx cached positions each, one token per sequence per step."""
+    import torch
+
+    mod = importlib.import_module("llm-inference-engine_b200")
+    mod.lib()
+    sz = SUM_NORM_SIZES[args.zasapel_size]
+    sz = dict(sz, window=0, moe=dict(sz["moe"], identity=0, shared=0))
+    W, H, M, R, rq, d, r = sz["width"], sz["heads"], sz["moe"], sz["rnn"], sz["q_rank"], sz["dim"], sz["rank"]
+    lb = LayerListBench(args, mod, args.ctx)
+    result = []
+    for build in (zasapel_model,) if args.no_closest else (zasapel_model, zefenex_model):
+        model, flops, n_bytes = build(lb, sz)
+        result.append(lb.measure(model.engine, flops, n_bytes))
+        del model
+        torch.cuda.empty_cache()
+    zasapel, closest = result[0], (result[1] if len(result) > 1 else None)
+    print(json.dumps({
+        "metric": "sum-norm model prefill / decode tokens/s", "value": zasapel["prefill"]["tokens_per_s"], "unit": "tokens/s (prefill)", "n_gpus": 1,
+        "steps": args.steps, "warmup": max(args.warmup, 3), "higher_is_better": True, "dtype": "bf16", "data": "synthetic", "impl": "b200",
+        "config": {"model": f"Zasapel-shaped, size {args.zasapel_size}: width {W}, layers minGRU / latent / latent / minGRU ({H} heads, dim {d}, rank {r}, query rank {rq}, "
+                            f"causal; the third reads the second's rows; state {R}), {sz['taps']} taps, dense ff {sz['dense_ff']} + 3 x {M['experts']} experts top {M['top']}",
+                   "closest": f"Zefenex-shaped: width {W}, 4 latent-attention layers ({H} heads, dim {d}+{sz['rot']}, rank {r}, causal), dense ff {sz['dense_ff']} + 3 x "
+                              f"{M['experts']} experts top {M['top']}",
+                   "prefill_tokens": lb.tokens, "decode_batch": lb.batch, "decode_context": args.ctx, "cache_policy": "weights larger than L2 at sizes m and l; no explicit flush"},
+        "zasapel": zasapel, "closest": closest,
         "e2e": "all numbers are taken through HybridDecoder.forward: host batch description in (one H2D copy per call), device logits out"}), flush=True)
 
 
@@ -1317,8 +1440,9 @@ def main():
     ap.add_argument("--latent-size", default="m", choices=list(LATENT_SIZES), help="--mode latent: which Zefenex-shaped model")
     ap.add_argument("--fedovik-size", default="m", choices=list(SHARED_NORM_SIZES), help="--mode fedovik: which Fedovik-shaped model")
     ap.add_argument("--silonex-size", default="m", choices=list(STREAM_SIZES), help="--mode silonex: which Silonex-shaped model")
-    ap.add_argument("--no-closest", action="store_true", help="--mode fedovik / silonex: leave out the closest other model beside it")
-    ap.add_argument("--mode", default="decode", choices=["decode", "prefill", "generate", "serve", "hybrid", "latent", "fedovik", "silonex"],
+    ap.add_argument("--zasapel-size", default="m", choices=list(SUM_NORM_SIZES), help="--mode zasapel: which Zasapel-shaped model")
+    ap.add_argument("--no-closest", action="store_true", help="--mode fedovik / silonex / zasapel: leave out the closest other model beside it")
+    ap.add_argument("--mode", default="decode", choices=["decode", "prefill", "generate", "serve", "hybrid", "latent", "fedovik", "silonex", "zasapel"],
                     help="decode (default, the BASELINE metric); prefill: one pass of --prefill-tokens tokens through all layers; generate: "
                          "the whole loop through b200_generate (prompt of --prefill-tokens tokens, --new-tokens sampled tokens, host in / host out)")
     ap.add_argument("--new-tokens", type=int, default=128)
@@ -1353,6 +1477,9 @@ def main():
         return
     if args.mode == "silonex":
         run_silonex(args)
+        return
+    if args.mode == "zasapel":
+        run_zasapel(args)
         return
     if args.mode == "fedovik":
         run_fedovik(args)

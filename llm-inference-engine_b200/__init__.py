@@ -107,6 +107,7 @@ ACT_RELU2, ACT_SILU, ACT_GELU_TANH, ACT_RELU, ACT_POLYNORM, ACT_CLAMP_GLU = 0, 1
  PLAN_MIXED_SAMPLE_ROWS) = range(16, 23)
 
 KV_PAGE_SIZE = 64
+MINGRU_SHORT = 8  # portions of fewer tokens take the minGRU's step kernel
 REQ_WAITING, REQ_RUNNING, REQ_FINISHED, REQ_REJECTED = 0, 1, 2, 3
 (PLAN_PREFILL_IDS, PLAN_PREFILL_LENS, PLAN_PREFILL_REQUESTS, PLAN_PREFILL_BLOCK_TABLE, PLAN_PREFILL_LAST_ROWS, PLAN_DECODE_TOKENS,
  PLAN_DECODE_STEPS, PLAN_DECODE_REQUESTS, PLAN_DECODE_BLOCK_TABLE) = range(9)
@@ -598,6 +599,32 @@ def moe_route_softmax(logits, bias, top):
     w = torch.empty((n, top), dtype=torch.float32, device=logits.device)
     check(lib().b200_moe_route_softmax(ptr(logits), logits.shape[1], ptr(bias), ptr(sel), ptr(w), n, logits.shape[1], top, stream()))
     return sel, w
+
+
+def poly_norm(x, coef, eps):
+    """In place on x [rows, cols]: coef[0] n(x) + coef[1] n(x^2) + coef[2] n(x^3) + coef[3], n(v) = v / rms(v) over the row."""
+    check(lib().b200_poly_norm(ptr(x), ptr(coef), float(eps), x.shape[0], x.shape[1], dtype_code(x), stream()))
+    return x
+
+
+def mingru(proj, bias, state, seq_start, seq_pos0, seq_slot, cols, chunk_tokens=64):
+    """proj [tokens, ld] (z | u | gate first), bias fp32 [2*cols] or None, state fp32 [slots, cols] (updated in place), host lists of the
+    portions -> out [tokens, cols]."""
+    torch = _torch()
+    n, dev = proj.shape[0], proj.device
+    chunks, n_short = [], 0
+    for s in range(len(seq_pos0)):
+        a, b = seq_start[s], seq_start[s + 1]
+        if b - a < MINGRU_SHORT:
+            n_short += b - a
+        else:
+            chunks += [[s, t, min(chunk_tokens, b - t), i] for i, t in enumerate(range(a, b, chunk_tokens))]
+    ints = [torch.tensor(v, dtype=torch.int32, device=dev) for v in (chunks or [[0, 0, 0, 0]], seq_start, seq_pos0, seq_slot)]
+    maps = torch.empty((max(len(chunks), 1), 2, cols), dtype=torch.float32, device=dev)
+    out = torch.empty((n, cols), dtype=proj.dtype, device=dev)
+    check(lib().b200_mingru(ptr(proj), proj.shape[1], ptr(bias), ptr(state), ptr(maps), ptr(out), ptr(ints[0]), len(chunks), ptr(ints[1]), ptr(ints[2]),
+                            ptr(ints[3]), len(seq_pos0), n_short, cols, dtype_code(proj), stream()))
+    return out
 
 
 def latent_prep_paged(proj, heads, dim, rot_dim, kv_rank, rot_dims, rot_base, kv_norm, eps, tok_seq, tok_pos, block_table, pool, t_pad, append=True):
