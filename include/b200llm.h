@@ -743,7 +743,7 @@ int b200_decay_recurrent(const float *rec, float *state, float *o, const int *se
 /* The minGRU recurrence (B200_MIXER_MINGRU).  proj [tokens, ld] of `dtype`: z | u | gate (cols each); bias fp32 [2*cols] for z and u, or
  * NULL; state fp32 [num_slots, cols]; out [tokens, cols] of `dtype`.  Portions of 8 tokens or more are described by `chunks`, DEVICE int4
  * {sequence, first packed row, tokens, index in its portion} (a portion's chunks in order and complete; 16-byte aligned); maps: fp32 scratch
- * [n_chunks, 2, cols].  n_short: tokens in shorter portions.  The other arrays are DEVICE arrays as in b200_hybrid_batch_t. */
+ * [n_chunks, 18, cols].  n_short: tokens in shorter portions.  The other arrays are DEVICE arrays as in b200_hybrid_batch_t. */
 int b200_mingru(const void *proj, int ld, const float *bias, float *state, float *maps, void *out, const int *chunks, int n_chunks,
                 const int *seq_start, const int *seq_pos0, const int *seq_slot, int n_seqs, int n_short, int cols, int dtype,
                 b200_stream_t stream);

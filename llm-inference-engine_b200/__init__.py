@@ -620,7 +620,7 @@ def mingru(proj, bias, state, seq_start, seq_pos0, seq_slot, cols, chunk_tokens=
         else:
             chunks += [[s, t, min(chunk_tokens, b - t), i] for i, t in enumerate(range(a, b, chunk_tokens))]
     ints = [torch.tensor(v, dtype=torch.int32, device=dev) for v in (chunks or [[0, 0, 0, 0]], seq_start, seq_pos0, seq_slot)]
-    maps = torch.empty((max(len(chunks), 1), 2, cols), dtype=torch.float32, device=dev)
+    maps = torch.empty((max(len(chunks), 1), 18, cols), dtype=torch.float32, device=dev)
     out = torch.empty((n, cols), dtype=proj.dtype, device=dev)
     check(lib().b200_mingru(ptr(proj), proj.shape[1], ptr(bias), ptr(state), ptr(maps), ptr(out), ptr(ints[0]), len(chunks), ptr(ints[1]), ptr(ints[2]),
                             ptr(ints[3]), len(seq_pos0), n_short, cols, dtype_code(proj), stream()))

@@ -36,6 +36,7 @@ namespace b200 {
 
 constexpr int kPageH = B200_KV_PAGE_SIZE;
 constexpr int kLatentPartTiles = 1184;     // (one-token tile, key share) pairs the partial-result scratch of the latent attention holds: 148 x 8
+constexpr int kMingruChunk = 128;  // tokens of one chunk of the minGRU's scan (longer portions: a multiple)
 constexpr int kLatentHeadsPerTile = 16;  // latent layers with at least this many heads run a decoded token's heads as one tensor-core tile
 static size_t align256(size_t v) { return (v + 255) & ~(size_t)255; }
 
@@ -708,6 +709,9 @@ struct b200_hybrid {
          *ys = nullptr, *lqn = nullptr, *lqr = nullptr, *lql = nullptr, *lol = nullptr, *lov = nullptr;
     float *lpart = nullptr, *rec = nullptr, *f32c = nullptr, *xs = nullptr;
     void *cat = nullptr, *xc = nullptr;
+    double *turns = nullptr;                    // the sinusoidal position vector's frequencies, formed by the first call after set_scratch
+    bool turns_ready = false;
+    float *maps = nullptr;
     int *meta = nullptr, *moe_i = nullptr;
     float *moe_f = nullptr;
     std::vector<int> host_meta;
@@ -716,7 +720,7 @@ struct b200_hybrid {
 namespace {
 
 struct Carve {
-    size_t x, f32a, f32b, xn, h, proj, mix, y, xg, u, yrows, us, ys, lqn, lqr, lql, lov, lpart, meta, moe_i, moe_f, rec, f32c, cat, xc, xs, total;
+    size_t x, f32a, f32b, xn, h, proj, mix, y, xg, u, yrows, us, ys, lqn, lqr, lql, lov, lpart, meta, moe_i, moe_f, rec, f32c, cat, xc, xs, turns, maps, total;
 };
 
 // rows of the input projection and columns of the output projection that ONE mixer owns
@@ -765,7 +769,7 @@ Carve carve(const b200_hybrid *m) {
     const b200_hybrid_config_t &c = m->cfg;
     const size_t T = (size_t)c.max_tokens, es = c.dtype == B200_F32 ? 4 : 2;
     size_t n_in = 1, n_mix = 1, n_f32 = 1, rows = 0, ff = 1, sff = 1, experts = 1, top = 1, lqn = 0, lqr = 0, lql = 0, lov = 0, lheads = 0, lpart = 0;
-    size_t n_rec = 0, n_heads = 0, n_cat = 0;
+    size_t n_rec = 0, n_heads = 0, n_cat = 0, n_gru = 0;
     bool pre_norm = false;
     const size_t t_pad = (T + 127) / 128 * 128;  // rows per head of the latent mixer's grouped GEMMs
     for (int i = 0; i < c.num_layers; ++i) {
@@ -787,6 +791,7 @@ Carve carve(const b200_hybrid *m) {
             }
             continue;
         }
+        if (l.mixer == B200_MIXER_MINGRU) n_gru = std::max(n_gru, (size_t)l.vdim);
         if (l.mixer == B200_MIXER_LATENT) {
             lqn = std::max(lqn, (size_t)l.heads * t_pad * l.dim), lqr = std::max(lqr, T * l.heads * l.rot_dim);
             lql = std::max(lql, (size_t)l.heads * t_pad * l.kv_rank), lov = std::max(lov, (size_t)l.heads * t_pad * l.vdim);
@@ -834,7 +839,9 @@ Carve carve(const b200_hybrid *m) {
     k.rec = align256(T * n_rec * 4), k.f32c = align256(2 * T * n_heads * 4), k.cat = align256(T * n_cat * es);
     k.xc = (c.loop_times > 0 && !pre_norm) ? align256(2 * T * c.width * es) : 0;
     k.xs = pre_norm ? align256(T * (size_t)std::max(c.streams, 1) * c.width * 4) : 0;
-    k.total = k.xs + k.x + k.f32a + k.f32b + k.xn + k.h + k.proj + 2 * k.mix + k.y + k.xg + k.u + k.yrows + k.us + k.ys + k.lqn + k.lqr + 2 * k.lql +
+    k.turns = c.pos_base > 0.0f ? align256((size_t)(c.width + 1) / 2 * 8) : 0;
+    k.maps = align256((T / kMingruChunk + (size_t)c.max_seqs) * kMingruMapRows * n_gru * 4);
+    k.total = k.maps + k.turns + k.xs + k.x + k.f32a + k.f32b + k.xn + k.h + k.proj + 2 * k.mix + k.y + k.xg + k.u + k.yrows + k.us + k.ys + k.lqn + k.lqr + 2 * k.lql +
               k.lov + k.lpart + k.meta + k.moe_i + k.moe_f + k.rec + k.f32c + k.cat + k.xc;
     return k;
 }
@@ -1059,6 +1066,8 @@ int b200_hybrid_set_scratch(b200_hybrid_t *m, void *ptr, size_t bytes) {
     m->cat = p, p += k.cat;
     m->xc = p, p += k.xc;
     m->xs = (float *)p, p += k.xs;
+    m->turns = (double *)p, p += k.turns, m->turns_ready = false;
+    m->maps = (float *)p, p += k.maps;
     return B200_OK;
 }
 
@@ -1192,10 +1201,10 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
     constexpr int kShortPortion = 8;
     static_assert(kShortPortion == kMingruShort, "one list of short portions serves both");
     int n_tiles = 0, n_short = 0, n_chunks = 0, gla_kinds = 0;
-    // minGRU chunks: at most 64 per portion (a chunk composes the maps of all chunks before it), of whole multiples of 64 tokens
+    // minGRU chunks: at most 64 per portion (a chunk composes the maps of all chunks before it), of whole multiples of kMingruChunk tokens
     int longest = 0;
     for (int s = 0; s < S; ++s) longest = std::max(longest, b->seq_start[s + 1] - b->seq_start[s]);
-    const int chunk_tokens = std::max(1, (longest + 4095) / 4096) * 64;
+    const int chunk_tokens = std::max(1, (longest + 64 * kMingruChunk - 1) / (64 * kMingruChunk)) * kMingruChunk;
     for (int s = 0; s < S; ++s) {
         const int t0 = b->seq_start[s], t1 = b->seq_start[s + 1];
         gla_kinds |= t1 - t0 == 1 ? kGlaOneToken : (t1 - t0 > 1 ? kGlaManyTokens : 0);
@@ -1482,8 +1491,12 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
         return more ? conv_input(next) : B200_OK;
     };
     if (sum_norm) {
-        RUN(launch_embed_pos(dt, d_ids, m->embedding, m->x, m->h, width, c.vocab, c.embed_scale != 0.0f ? c.embed_scale : 1.0f, c.pos_base, ring_conv(0, 0),
-                             one_token, pm, NT, st));
+        if (c.pos_base > 0.0f && !m->turns_ready) {
+            RUN(launch_pos_turns(m->turns, width, c.pos_base, st));
+            m->turns_ready = true;
+        }
+        RUN(launch_embed_pos(dt, d_ids, m->embedding, m->x, m->h, width, c.vocab, c.embed_scale != 0.0f ? c.embed_scale : 1.0f, c.pos_base > 0.0f ? m->turns : nullptr,
+                             ring_conv(0, 0), one_token, pm, NT, st));
         RUN(conv_input(ring_conv(0, 0)));
     }
 
@@ -1597,7 +1610,7 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
             RUN(launch_latent_gate(dt, m->lov, gate, lp.n_in, m->mix2, NT, t_pad, l.heads, l.vdim, st, l.head_gate));
             n_mixed = hv;
         } else if (l.mixer == B200_MIXER_MINGRU) {
-            RUN(launch_mingru(dt, m->proj, lp.n_in, l.b_in, (float *)(m->state_pool + lp.state_off), m->f32a, m->mix2, d_chunks, n_chunks, d_start, d_pos0,
+            RUN(launch_mingru(dt, m->proj, lp.n_in, l.b_in, (float *)(m->state_pool + lp.state_off), m->maps, m->mix2, d_chunks, n_chunks, d_start, d_pos0,
                               d_slot, S, n_short, l.vdim, st));
             n_mixed = l.vdim;
         } else {

@@ -114,14 +114,16 @@ struct PortionMap { const int *tok_seq, *tok_pos, *seq_start, *seq_pos0, *seq_sl
 int launch_sum_norm(int dtype, float *x, const void *y_dense, const void *y_rows, const int *pair_row, int top, const void *y_shared,
                     const float *shared_gate, float alpha, const float *g, float eps, int width, float *trace, void *h_out, RingConv own, RingConv next,
                     int one_token, PortionMap pm, int tokens, cudaStream_t st);
-int launch_embed_pos(int dtype, const int *ids, const void *table, float *x, void *h_out, int width, int vocab, float scale, float base, RingConv next,
-                     int one_token, PortionMap pm, int tokens, cudaStream_t st);
+// turns: fp64 [(width + 1) / 2], written once by launch_pos_turns; NULL: no position vector
+int launch_pos_turns(double *turns, int width, float base, cudaStream_t st);
+int launch_embed_pos(int dtype, const int *ids, const void *table, float *x, void *h_out, int width, int vocab, float scale, const double *turns,
+                     RingConv next, int one_token, PortionMap pm, int tokens, cudaStream_t st);
 int launch_conv_input(int dtype, const float *x, void *h, int width, RingConv cv, PortionMap pm, int tokens, cudaStream_t st);
 
 // mingru.cu: proj row z | u | gate (cols each), bias [2 * cols] or NULL, state fp32 [slots, cols]; out [tokens, cols].  Portions of at least
 // kMingruShort tokens arrive as chunks, int4 {sequence, first packed row, tokens, index in its portion}, a portion's chunks in order; maps: fp32
-// scratch [n_chunks, 2, cols].  n_short: tokens in shorter portions (0: their kernel is not launched)
-constexpr int kMingruShort = 8;
+// scratch [n_chunks, kMingruMapRows, cols].  n_short: tokens in shorter portions (0: their kernel is not launched)
+constexpr int kMingruShort = 8, kMingruMapRows = 18;
 int launch_mingru(int dtype, const void *proj, int ld, const float *bias, float *state, float *maps, void *out, const int *chunks, int n_chunks,
                   const int *seq_start, const int *seq_pos0, const int *seq_slot, int n_seqs, int n_short, int cols, cudaStream_t st);
 

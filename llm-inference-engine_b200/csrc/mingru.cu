@@ -2,10 +2,13 @@
 //     s_t = (1 - z_t) s_(t-1) + z_t c_t,   z = sigmoid(z-in + b_z),   u = u-in + b_u,   c = u + 1/2 where u >= 0, sigmoid(u) elsewhere,
 // result s_t * silu(gate_t).  The state is one fp32 vector per sequence; everything from the projections' outputs on is fp32.
 //
-// A step is an affine map s -> A s + B with A = 1 - z, B = z c, and maps compose, so a long portion is not a chain of its tokens: it is cut
-// into chunks, every chunk's composed map is formed on its own (mingru_chunk_kernel), and mingru_apply_kernel composes the maps of the
-// chunks before its own and then walks its tokens.  The first chunk's map has the sequence's state already applied (B = state after the
-// chunk), and its A entry carries the state the chunk starts from: the state slot is read by one kernel and written by the next.
+// A step is an affine map s -> A s + B with A = 1 - z, B = z c, and maps compose, so a long portion is not a chain of its tokens.  It is cut
+// into chunks and every chunk into kSubs runs of tokens, one per warp of a CTA (a lane holds N adjacent channels):
+//   * mingru_chunk_kernel forms the map of every run and, composed, of every chunk;
+//   * mingru_apply_kernel composes the maps of the chunks before its own (shared out over its warps) and of the runs before each warp's, and
+//     walks the tokens.
+// The first chunk's map has the sequence's state already applied (its B is the state after the chunk), and its A entry carries the state the
+// chunk starts from: the state slot is read by one kernel and written by the next.
 // Portions of fewer than kMingruShort tokens (decoded tokens) are walked by one thread per channel in mingru_step_kernel.
 #include "hybrid_ops.cuh"
 
@@ -42,57 +45,111 @@ struct MingruCols {
     __device__ __forceinline__ void gate(int t, float *g) const { load_n<T, N>(proj + (size_t)t * ld + 2 * cols + col, g); }
 };
 
-// grid (channel blocks, chunks)
+// maps: fp32 [chunks, 1 + kSubs, 2 (A, B), cols]: the chunk's map, then its runs'
+constexpr int kSubs = 8;
+static_assert((1 + kSubs) * 2 == kMingruMapRows, "the scratch of the chunk maps");
+
+// grid (blocks of 32 * N channels, chunks)
 template <typename T, int N>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(32 * kSubs)
 mingru_chunk_kernel(const T *__restrict__ proj, int ld, const float *__restrict__ bias, const float *__restrict__ state, float *__restrict__ maps,
                     const int4 *__restrict__ chunks, const int *__restrict__ seq_pos0, const int *__restrict__ seq_slot, int cols) {
-    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * N;
-    if (c >= cols) return;
+    __shared__ float sa[kSubs][32 * N], sb[kSubs][32 * N];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, c = (blockIdx.x * 32 + lane) * N;
     const int4 ch = chunks[blockIdx.y];  // sequence, first packed row, tokens, index in its portion
-    const MingruCols<T, N> in(proj, ld, cols, bias, c);
-    float A[N], B[N], first[N];
+    const int run = (ch.z + kSubs - 1) / kSubs, t0 = ch.y + min(ch.z, warp * run), t1 = ch.y + min(ch.z, (warp + 1) * run);
+    float *m = maps + (size_t)blockIdx.y * (1 + kSubs) * 2 * cols + c;
+    float A[N], B[N];
 #pragma unroll
-    for (int i = 0; i < N; ++i) A[i] = 1.0f, B[i] = first[i] = 0.0f;
+    for (int i = 0; i < N; ++i) A[i] = 1.0f, B[i] = 0.0f;
+    if (c < cols) {
+        const MingruCols<T, N> in(proj, ld, cols, bias, c);
+#pragma unroll 8
+        for (int t = t0; t < t1; ++t) {
+            float z[N], u[N];
+            in.load(t, z, u);
+#pragma unroll
+            for (int i = 0; i < N; ++i) {
+                const MingruStep s = mingru_step(z[i], u[i]);
+                A[i] *= s.keep, B[i] = fmaf(s.keep, B[i], s.add);
+            }
+        }
+        store_n<float, N>(m + (size_t)(1 + warp) * 2 * cols, A);
+        store_n<float, N>(m + (size_t)(1 + warp) * 2 * cols + cols, B);
+    }
+#pragma unroll
+    for (int i = 0; i < N; ++i) sa[warp][lane * N + i] = A[i], sb[warp][lane * N + i] = B[i];
+    __syncthreads();
+    if (warp > 0 || c >= cols) return;
+    float first[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) first[i] = 0.0f;
     if (ch.w == 0 && seq_pos0[ch.x] > 0) load_n<float, N>(state + (size_t)seq_slot[ch.x] * cols + c, first);
 #pragma unroll
-    for (int i = 0; i < N; ++i) B[i] = first[i];
-#pragma unroll 8
-    for (int t = ch.y; t < ch.y + ch.z; ++t) {
-        float z[N], u[N];
-        in.load(t, z, u);
+    for (int i = 0; i < N; ++i) {
+        A[i] = 1.0f, B[i] = first[i];
 #pragma unroll
-        for (int i = 0; i < N; ++i) {
-            const MingruStep s = mingru_step(z[i], u[i]);
-            A[i] *= s.keep, B[i] = fmaf(s.keep, B[i], s.add);
+        for (int w = 0; w < kSubs; ++w) {
+            const float a = sa[w][lane * N + i];
+            A[i] *= a, B[i] = fmaf(a, B[i], sb[w][lane * N + i]);
         }
     }
-    float *m = maps + (size_t)blockIdx.y * 2 * cols + c;
     store_n<float, N>(m, ch.w == 0 ? first : A);
     store_n<float, N>(m + cols, B);
 }
 
 template <typename T, int N>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(32 * kSubs)
 mingru_apply_kernel(const T *__restrict__ proj, int ld, const float *__restrict__ bias, float *__restrict__ state, const float *__restrict__ maps,
                     T *__restrict__ out, const int4 *__restrict__ chunks, const int *__restrict__ seq_start, const int *__restrict__ seq_slot, int cols) {
-    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * N;
-    if (c >= cols) return;
+    __shared__ float sa[kSubs][32 * N], sb[kSubs][32 * N];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, c = (blockIdx.x * 32 + lane) * N;
     const int4 ch = chunks[blockIdx.y];
-    const MingruCols<T, N> in(proj, ld, cols, bias, c);
-    const float *m0 = maps + (size_t)(blockIdx.y - ch.w) * 2 * cols + c;
+    const bool live = c < cols;
+    const size_t per = (size_t)(1 + kSubs) * 2 * cols;
+    const float *m0 = maps + (size_t)(blockIdx.y - ch.w) * per + c, *own = maps + (size_t)blockIdx.y * per + 2 * cols + c;
     float s[N];
-    load_n<float, N>(ch.w == 0 ? m0 : m0 + cols, s);
-#pragma unroll 8
-    for (int k = 1; k < ch.w; ++k) {
-        float A[N], B[N];
-        load_n<float, N>(m0 + (size_t)k * 2 * cols, A);
-        load_n<float, N>(m0 + (size_t)k * 2 * cols + cols, B);
 #pragma unroll
-        for (int i = 0; i < N; ++i) s[i] = fmaf(A[i], s[i], B[i]);
+    for (int i = 0; i < N; ++i) s[i] = 0.0f;
+    if (live) load_n<float, N>(ch.w == 0 ? m0 : m0 + cols, s);
+    if (ch.w > 1) {  // the chunks 1 .. ch.w - 1 (the whole CTA agrees)
+        const int share = (ch.w - 1 + kSubs - 1) / kSubs, k0 = 1 + warp * share, k1 = min(ch.w, k0 + share);
+        float A[N], B[N];
+#pragma unroll
+        for (int i = 0; i < N; ++i) A[i] = 1.0f, B[i] = 0.0f;
+        if (live) {
+#pragma unroll 4
+            for (int k = k0; k < k1; ++k) {
+                float a[N], b[N];
+                load_n<float, N>(m0 + k * per, a);
+                load_n<float, N>(m0 + k * per + cols, b);
+#pragma unroll
+                for (int i = 0; i < N; ++i) A[i] *= a[i], B[i] = fmaf(a[i], B[i], b[i]);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < N; ++i) sa[warp][lane * N + i] = A[i], sb[warp][lane * N + i] = B[i];
+        __syncthreads();
+#pragma unroll
+        for (int w = 0; w < kSubs; ++w)
+#pragma unroll
+            for (int i = 0; i < N; ++i) s[i] = fmaf(sa[w][lane * N + i], s[i], sb[w][lane * N + i]);
     }
+    if (!live) return;
+    const MingruCols<T, N> in(proj, ld, cols, bias, c);
+#pragma unroll
+    for (int w = 0; w < kSubs - 1; ++w) {
+        if (w < warp) {
+            float a[N], b[N];
+            load_n<float, N>(own + (size_t)w * 2 * cols, a);
+            load_n<float, N>(own + (size_t)w * 2 * cols + cols, b);
+#pragma unroll
+            for (int i = 0; i < N; ++i) s[i] = fmaf(a[i], s[i], b[i]);
+        }
+    }
+    const int run = (ch.z + kSubs - 1) / kSubs, t0 = ch.y + min(ch.z, warp * run), t1 = ch.y + min(ch.z, (warp + 1) * run);
 #pragma unroll 8
-    for (int t = ch.y; t < ch.y + ch.z; ++t) {
+    for (int t = t0; t < t1; ++t) {
         float z[N], u[N], g[N];
         in.load(t, z, u);
         in.gate(t, g);
@@ -104,7 +161,7 @@ mingru_apply_kernel(const T *__restrict__ proj, int ld, const float *__restrict_
         }
         store_n<T, N>(out + (size_t)t * cols + c, g);
     }
-    if (ch.y + ch.z == seq_start[ch.x + 1]) store_n<float, N>(state + (size_t)seq_slot[ch.x] * cols + c, s);
+    if (t1 > t0 && t1 == seq_start[ch.x + 1]) store_n<float, N>(state + (size_t)seq_slot[ch.x] * cols + c, s);
 }
 
 // grid (channel blocks, sequences): portions of fewer than kMingruShort tokens
@@ -148,8 +205,9 @@ int launch_mingru(int dtype, const void *proj, int ld, const float *bias, float 
         if (n_chunks > 0) {
             auto chunk = vec ? mingru_chunk_kernel<T, 4> : mingru_chunk_kernel<T, 1>;
             auto apply = vec ? mingru_apply_kernel<T, 4> : mingru_apply_kernel<T, 1>;
-            chunk<<<dim3(blocks, n_chunks), threads, 0, st>>>((const T *)proj, ld, bias, state, maps, ch, seq_pos0, seq_slot, cols);
-            apply<<<dim3(blocks, n_chunks), threads, 0, st>>>((const T *)proj, ld, bias, state, maps, (T *)out, ch, seq_start, seq_slot, cols);
+            const dim3 grid((cols + 32 * n - 1) / (32 * n), n_chunks);
+            chunk<<<grid, 32 * kSubs, 0, st>>>((const T *)proj, ld, bias, state, maps, ch, seq_pos0, seq_slot, cols);
+            apply<<<grid, 32 * kSubs, 0, st>>>((const T *)proj, ld, bias, state, maps, (T *)out, ch, seq_start, seq_slot, cols);
         }
         if (n_short > 0) {
             auto step = vec ? mingru_step_kernel<T, 4> : mingru_step_kernel<T, 1>;

@@ -159,35 +159,47 @@ sum_norm_kernel(float *x, const T *__restrict__ y_dense, const T *__restrict__ y
     }
 }
 
-// x[t, :] = table[id] * scale (+ the sinusoidal position vector: channels 2i, 2i + 1 receive sin, cos of p * base^(-2i / width)); h_out as
-// above.  A CTA takes `run` consecutive rows, so a thread forms the frequency of a channel once.  The angle is taken in turns, in fp64, and
-// only its fraction goes to fp32: exact to the last bit of sin / cos at any position.
-template <typename T>
+// turns[i] = base^(-2i / width) / (2 pi): turns per position of channels 2i and 2i + 1
+__global__ void pos_turns_kernel(double *__restrict__ turns, int width, float base) {
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (2 * i < width) turns[i] = exp2(-2.0 * (double)i / (double)width * log2((double)base)) * 0.15915494309189533577;
+}
+
+// x[t, :] = table[id] * scale (+ the sinusoidal position vector: channels 2i, 2i + 1 receive sin, cos of p * base^(-2i / width); turns NULL:
+// none); h_out as above.  The angle is taken in turns, in fp64, and only its fraction goes to fp32, so that a far position costs no bits.
+// grid (tokens, channel blocks); N = 1 or 4 channels per thread.
+template <typename T, int N>
 __global__ void __launch_bounds__(256)
 embed_pos_kernel(const int *__restrict__ ids, const T *__restrict__ table, float *__restrict__ x, T *__restrict__ h_out, int width, int vocab,
-                 float scale, float base, int tokens, int run, RingConv next, int one_token, PortionMap pm) {
-    const int t0 = blockIdx.x * run, t1 = min(tokens, t0 + run);
-    const bool conv = h_out && one_token && next.taps > 0;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) {
-        const double turns = base > 0.0f ? exp2(-(double)(c & ~1) / (double)width * log2((double)base)) * 0.15915494309189533577 : 0.0;
-        for (int t = t0; t < t1; ++t) {
-            int id = ids[t];
-            id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);  // the host has refused ids outside the vocabulary
-            float v = Elem<T>::to_f(table[(size_t)id * width + c]) * scale;
-            const int pos = pm.tok_pos[t];
-            if (base > 0.0f) {
-                const double a = (double)pos * turns;
-                const float half_turns = 2.0f * (float)(a - rint(a));
-                v += (c & 1) ? cospif(half_turns) : sinpif(half_turns);
-            }
-            x[(size_t)t * width + c] = v;
-            if (conv) {
-                const int slot = pm.seq_slot[pm.tok_seq[t]];
-                conv_from_ring<1>(&v, c, width, pos, next.taps > 1 ? next.ring + (size_t)slot * (next.taps - 1) * width : nullptr, next.w, next.taps);
-            }
-            if (h_out && (conv || next.taps == 0)) h_out[(size_t)t * width + c] = Elem<T>::from_f(v);
+                 float scale, const double *__restrict__ turns, RingConv next, int one_token, PortionMap pm) {
+    const int t = blockIdx.x, c = (blockIdx.y * blockDim.x + threadIdx.x) * N;
+    if (c >= width) return;
+    int id = ids[t];
+    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);  // the host has refused ids outside the vocabulary
+    const int pos = pm.tok_pos[t];
+    float v[N];
+    load_n<T, N>(table + (size_t)id * width + c, v);
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] *= scale;
+    if (turns) {
+#pragma unroll
+        for (int i = 0; i < N; i += 2) {
+            const double a = (double)pos * turns[(c + i) >> 1];
+            float sn, cn;
+            sincospif(2.0f * (float)(a - rint(a)), &sn, &cn);
+            if constexpr (N == 1) v[0] += (c & 1) ? cn : sn;
+            else v[i] += sn, v[i + 1] += cn;
         }
     }
+    store_n<float, N>(x + (size_t)t * width + c, v);
+    if (!h_out) return;
+    if (one_token && next.taps > 0) {
+        const int slot = pm.seq_slot[pm.tok_seq[t]];
+        conv_from_ring<N>(v, c, width, pos, next.taps > 1 ? next.ring + (size_t)slot * (next.taps - 1) * width : nullptr, next.w, next.taps);
+    } else if (next.taps > 0) {
+        return;
+    }
+    store_n<T, N>(h_out + (size_t)t * width + c, v);
 }
 
 // h[t, :] = T(x[t, :] + conv(x)[t, :]).  grid (runs of kConvRun packed rows, channel blocks); N channels per thread.  TAPS: taps at compile
@@ -279,13 +291,21 @@ int launch_sum_norm(int dtype, float *x, const void *y_dense, const void *y_rows
     return cuda_status("sum_norm launch");
 }
 
-int launch_embed_pos(int dtype, const int *ids, const void *table, float *x, void *h_out, int width, int vocab, float scale, float base, RingConv next,
-                     int one_token, PortionMap pm, int tokens, cudaStream_t st) {
+int launch_pos_turns(double *turns, int width, float base, cudaStream_t st) {
+    pos_turns_kernel<<<(width + 511) / 512, 256, 0, st>>>(turns, width, base);
+    return cuda_status("pos_turns launch");
+}
+
+int launch_embed_pos(int dtype, const int *ids, const void *table, float *x, void *h_out, int width, int vocab, float scale, const double *turns,
+                     RingConv next, int one_token, PortionMap pm, int tokens, cudaStream_t st) {
     if (tokens == 0) return B200_OK;
-    const int run = tokens >= 148 * 8 ? 8 : 1;
     B200_DISPATCH_DTYPE(dtype, {
-        embed_pos_kernel<T><<<(tokens + run - 1) / run, 256, 0, st>>>(ids, (const T *)table, x, (T *)h_out, width, vocab, scale, base, tokens, run, next,
-                                                                      one_token, pm);
+        const bool vec = width % 4 == 0 && all_aligned16({table, x, h_out, next.ring, next.w});
+        const int cols = vec ? width / 4 : width;
+        const int threads = std::min(256, (cols + 31) / 32 * 32);
+        auto kern = vec ? embed_pos_kernel<T, 4> : embed_pos_kernel<T, 1>;
+        kern<<<dim3(tokens, (cols + threads - 1) / threads), threads, 0, st>>>(ids, (const T *)table, x, (T *)h_out, width, vocab, scale, turns, next,
+                                                                               one_token, pm);
     });
     return cuda_status("embed_pos launch");
 }
