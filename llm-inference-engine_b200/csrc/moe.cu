@@ -14,6 +14,7 @@
 #include "hybrid_ops.cuh"
 
 #include <algorithm>
+#include <type_traits>
 
 namespace b200 {
 
@@ -267,17 +268,25 @@ __global__ void bias_activation_kernel(T *__restrict__ x, const float *__restric
 // In place, one CTA per row: x = a n(x) + b n(x^2) + c n(x^3) + e, n(v) = v / sqrt(mean over the row of v^2 + eps).  One pass forms the three
 // mean squares (of x, x^2 and x^3) together; a thread's pieces stay in registers in between when the row is short enough.
 template <typename T, bool VEC>
-__global__ void __launch_bounds__(512)
+__global__ void __launch_bounds__(256)
 poly_norm_kernel(T *__restrict__ x, const float *__restrict__ coef, float eps, int cols) {
-    constexpr int N = VEC ? Elem<T>::kVec : 1, KP = VEC ? 2 : 8;
-    __shared__ float red[3][17];
+    constexpr int N = VEC ? Elem<T>::kVec : 1, KP = VEC ? 4 : 8;
+    __shared__ float red[3][9];
     T *row = x + (size_t)blockIdx.x * cols;
-    auto load = [&](int c, float *v) {
-        if constexpr (VEC) unpack16<T>(ld_v4(row + c), v);
-        else v[0] = Elem<T>::to_f(row[c]);
+    // a piece as it lies in memory: 16 bytes, or one element
+    using Piece = typename std::conditional<VEC, uint4, T>::type;
+    auto load = [&](int c) -> Piece {
+        if constexpr (VEC) return ld_v4(row + c);
+        else return row[c];
+    };
+    auto open = [&](const Piece &p, float *v) {
+        if constexpr (VEC) unpack16<T>(p, v);
+        else v[0] = Elem<T>::to_f(p);
     };
     float s1 = 0.0f, s2 = 0.0f, s3 = 0.0f;
-    auto add = [&](const float *v) {
+    auto add = [&](const Piece &p) {
+        float v[N];
+        open(p, v);
 #pragma unroll
         for (int i = 0; i < N; ++i) {
             const float q = v[i] * v[i];
@@ -285,18 +294,18 @@ poly_norm_kernel(T *__restrict__ x, const float *__restrict__ coef, float eps, i
         }
     };
     const bool held = cols <= (int)blockDim.x * N * KP;
-    float keep[KP][N];
+    Piece keep[KP];
     if (held) {
 #pragma unroll
         for (int i = 0; i < KP; ++i) {
             const int c = (threadIdx.x + i * blockDim.x) * N;
-            if (c < cols) load(c, keep[i]), add(keep[i]);
+            if (c < cols) keep[i] = load(c);
         }
+#pragma unroll
+        for (int i = 0; i < KP; ++i)
+            if ((threadIdx.x + i * blockDim.x) * N < cols) add(keep[i]);
     } else {
-        for (int c = threadIdx.x * N; c < cols; c += blockDim.x * N) {
-            float v[N];
-            load(c, v), add(v);
-        }
+        for (int c = threadIdx.x * N; c < cols; c += blockDim.x * N) add(load(c));
     }
     s1 = warp_sum(s1), s2 = warp_sum(s2), s3 = warp_sum(s3);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
@@ -306,7 +315,9 @@ poly_norm_kernel(T *__restrict__ x, const float *__restrict__ coef, float eps, i
     for (int w = 0; w < nwarp; ++w) s1 += red[0][w], s2 += red[1][w], s3 += red[2][w];
     const float n = (float)cols;
     const float a = coef[0] * rsqrtf(s1 / n + eps), b = coef[1] * rsqrtf(s2 / n + eps), d = coef[2] * rsqrtf(s3 / n + eps), e0 = coef[3];
-    auto finish = [&](int c, float *v) {
+    auto finish = [&](int c, const Piece &p) {
+        float v[N];
+        open(p, v);
 #pragma unroll
         for (int i = 0; i < N; ++i) v[i] = fmaf(v[i], fmaf(v[i], fmaf(v[i], d, b), a), e0);
         if constexpr (VEC) st_v4(row + c, pack16<T>(v));
@@ -320,10 +331,7 @@ poly_norm_kernel(T *__restrict__ x, const float *__restrict__ coef, float eps, i
         }
         return;
     }
-    for (int c = threadIdx.x * N; c < cols; c += blockDim.x * N) {
-        float v[N];
-        load(c, v), finish(c, v);
-    }
+    for (int c = threadIdx.x * N; c < cols; c += blockDim.x * N) finish(c, load(c));
 }
 
 // SIMT grouped GEMM, 64 x 64 tile, fp32 accumulation.  The tensor-core path of the dense linears does not apply: an expert's rows are
@@ -544,7 +552,7 @@ int launch_poly_norm(int dtype, void *x, const float *coef, float eps, int rows,
     B200_DISPATCH_DTYPE(dtype, {
         const bool vec = cols % Elem<T>::kVec == 0 && (reinterpret_cast<size_t>(x) & 15) == 0;
         const int per = vec ? Elem<T>::kVec : 1;
-        const int threads = std::min(512, std::max(32, ((cols + per - 1) / per + 31) / 32 * 32));
+        const int threads = std::min(256, std::max(32, ((cols + per - 1) / per + 31) / 32 * 32));
         auto kern = vec ? poly_norm_kernel<T, true> : poly_norm_kernel<T, false>;
         kern<<<rows, threads, 0, st>>>((T *)x, coef, eps, cols);
     });
