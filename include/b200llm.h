@@ -488,7 +488,7 @@ typedef struct {
     int max_pages_per_seq;
     float embed_scale;  /* x = embedding[token] * embed_scale; 0 reads as 1                                                           */
     float logit_softcap;/* logits <- cap * tanh(logits / cap); 0: none                                                                */
-    int final_norm;     /* b200_norm_kind_t of the model's last norm (RMS_POST: plain RMS norm; DYT: packed [w | b | alpha];
+    int final_norm;     /* b200_norm_kind_t of the model's last norm (RMS_POST, RMS_SUM: RMS norm; DYT: packed [w | b | alpha];
                            LN_PARALLEL: layer norm, packed [w | b])                                                                  */
     int loop_start, loop_stop, loop_times; /* loop_times > 0: layers [loop_start, loop_stop) run loop_times times in a row with the same
                            weights, every pass with a cache and state of its own (b200_hybrid_set_loop gives the entry step's weights);
