@@ -468,10 +468,11 @@ typedef enum {
                                     every mixer has an output projection of its own (w_out; side->w_out); with branch_norm set, the
                                     mixer sublayer's result is mix_scale * rmsnorm(mixer) * branch_norm + side_scale * rmsnorm(side) *
                                     side->branch_norm.  Feed-forward: DENSE, gated (w_up [2*expert_ff, width]: gate rows, then up rows) */
-    B200_NORM_RMS_SUM = 4        /* the norm takes the SUM: x <- rmsnorm(residual_scale * x + mixer(x')) * norm1, then the same with the
+    B200_NORM_RMS_SUM = 4,       /* the norm takes the SUM: x <- rmsnorm(residual_scale * x + mixer(x')) * norm1, then the same with the
                                     feed-forward and norm2.  A sublayer reads x' = x + conv(x), a causal convolution over time on every
                                     channel (in_taps, in_conv1 / in_conv2; in_taps == 0: x' = x); its last in_taps - 1 inputs are
                                     part of a sequence's state                                                                        */
+    B200_NORM_LN_POST = 5        /* x += branch_scale * layernorm(sublayer(x)) * norm1 / norm2 (weight, no bias)                      */
 } b200_norm_kind_t;
 typedef enum {
     B200_ROUTE_SIGMOID = 0,      /* scores = sigmoid(logits), the chosen scores are the weights, applied to the expert's INPUT        */
@@ -489,7 +490,7 @@ typedef struct {
     float embed_scale;  /* x = embedding[token] * embed_scale; 0 reads as 1                                                           */
     float logit_softcap;/* logits <- cap * tanh(logits / cap); 0: none                                                                */
     int final_norm;     /* b200_norm_kind_t of the model's last norm (RMS_POST, RMS_SUM: RMS norm; DYT: packed [w | b | alpha];
-                           LN_PARALLEL: layer norm, packed [w | b])                                                                  */
+                           LN_PARALLEL, LN_PRE: layer norm, packed [w | b]; LN_POST: layer norm, weight only)                        */
     int loop_start, loop_stop, loop_times; /* loop_times > 0: layers [loop_start, loop_stop) run loop_times times in a row with the same
                            weights, every pass with a cache and state of its own (b200_hybrid_set_loop gives the entry step's weights);
                            0: every layer runs once                                                                                  */
@@ -498,13 +499,14 @@ typedef struct {
     float pos_base;     /* RMS_SUM layers: > 0: a sinusoidal position vector joins the embedding: channels 2i, 2i + 1 receive sin, cos of
                            p * pos_base^(-2i / width); 0: none                                                                        */
     float residual_scale; /* RMS_SUM layers: see B200_NORM_RMS_SUM                                                                    */
+    float branch_scale; /* LN_POST layers: see B200_NORM_LN_POST                                                                      */
 } b200_hybrid_config_t;
 
 typedef struct b200_hybrid_layer_s {
     int mixer;          /* b200_mixer_kind_t                                                                                          */
     int heads, kv_heads, dim, vdim;
     float scale;        /* ATTN, LATENT: score scale                                                                                  */
-    int chunk;          /* ATTN: position i sees j <= i with floor(i/chunk) == floor(j/chunk); 0 = plain causal                       */
+    int chunk;          /* ATTN, ATTN_SCORED: position i sees j <= i with floor(i/chunk) == floor(j/chunk); 0 = plain causal                       */
     float tau;          /* GLA: decay = sigmoid(z)^(1/tau)                                                                            */
     int decay_rank;     /* GLA: inner size of the low-rank decay projection                                                           */
     int mlp;            /* b200_mlp_kind_t                                                                                            */
@@ -516,7 +518,7 @@ typedef struct b200_hybrid_layer_s {
                            gate (heads*vdim) and, unless kv_from >= 0, the down-projection (kv_rank + rot_dim).  K = width            */
     const void *w_out;  /* [width, heads*vdim]                                                                                        */
     const float *q_norm, *k_norm; /* ATTN: [heads*dim], [kv_heads*dim]: RMS norm over the WHOLE projection                            */
-    const float *sink;  /* ATTN, LATENT: [heads] or NULL                                                                              */
+    const float *sink;  /* ATTN, LATENT, ATTN_SCORED with softmax weights: [heads] or NULL                                            */
     const void *w_decay; const float *decay_bias; /* GLA: [heads*dim, decay_rank], [heads*dim]                                        */
     const float *out_norm;        /* GLA: [vdim], shared by the heads                                                                 */
     const float *norm1, *norm2;   /* RMS_POST: [width]                                                                                */
@@ -592,13 +594,24 @@ typedef struct b200_hybrid_layer_s {
     /* ---- LATENT with q_rank > 0: queries through a normed low-rank row of their own: w_in rows dq (q_rank), then (kv_from < 0) the
      *      down-projection (kv_rank + rot_dim), then the gate; q = w_uq (rmsnorm(dq) * dq_norm) */
     int q_rank;
-    int head_gate;                /* 1: ONE gate per head (heads rows) instead of one per value channel                               */
+    int head_gate;                /* LATENT: 1: ONE gate per head (heads rows) instead of one per value channel; 2: no gate, no rows for it */
     const float *dq_norm;         /* [q_rank]                                                                                         */
     const void *w_uq;             /* [heads*(dim + rot_dim), q_rank]                                                                  */
     /* ---- MINGRU: heads = dim = 1, vdim = state size; w_in rows z, u, gate (vdim each); b_in [2*vdim] for z and u                   */
     /* ---- activations with parameters */
     const float *act_coef;        /* POLYNORM: [4] a, b, c, e                                                                         */
     float act_limit, act_slope;   /* CLAMP_GLU; act_limit <= 0: no clamp                                                              */
+    /* ---- ATTN_SCORED: a linear distance bias, and values that carry a share of an earlier layer's values of the same token */
+    const float *dist_slope;      /* [heads] or NULL: score(i, j) -= dist_slope * (i - j)                                             */
+    int v_share;                  /* 1: this layer's values (as projected) are kept for the rest of the call; 2: v <- (1 - v_lambda) v +
+                                     v_lambda * (the kept values), before the values are cached; 0: neither                           */
+    float v_lambda;
+    /* ---- LATENT: other rotations of the rotated part */
+    int rot_pairs;                /* 1: the rotating pairs are (2i, 2i+1) instead of (i, i + rot_dims/2)                              */
+    const double *rot_turns;      /* DEVICE [rot_dims/2]: turns per position of every pair (frequency / 2 pi), in place of rot_base; or NULL */
+    float rot_amp;                /* cosine and sine are multiplied by this; 0 reads as 1                                             */
+    /* ---- MOE, SOFTMAX */
+    const float *logit_bias;      /* [experts + identity] added to the router's logits, or NULL                                       */
 } b200_hybrid_layer_t;
 
 typedef struct {

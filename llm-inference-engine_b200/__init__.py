@@ -63,7 +63,7 @@ class HybridConfig(C.Structure):
     _fields_ = [("width", C.c_int), ("vocab", C.c_int), ("num_layers", C.c_int), ("dtype", C.c_int), ("norm_eps", C.c_float),
                 ("max_tokens", C.c_int), ("max_seqs", C.c_int), ("max_pages_per_seq", C.c_int), ("embed_scale", C.c_float),
                 ("logit_softcap", C.c_float), ("final_norm", C.c_int), ("loop_start", C.c_int), ("loop_stop", C.c_int), ("loop_times", C.c_int),
-                ("logit_scale", C.c_float), ("streams", C.c_int), ("pos_base", C.c_float), ("residual_scale", C.c_float)]
+                ("logit_scale", C.c_float), ("streams", C.c_int), ("pos_base", C.c_float), ("residual_scale", C.c_float), ("branch_scale", C.c_float)]
 
 
 class HybridLayer(C.Structure):
@@ -88,7 +88,9 @@ class HybridLayer(C.Structure):
                 ("v_norm", C.c_int), ("softcap", C.c_float), ("gate_act", C.c_int), ("conv_b", C.c_void_p), ("skip", C.c_void_p),
                 ("norm_groups", C.c_int), ("head_decay", C.c_void_p), ("hc1", C.c_void_p), ("hc2", C.c_void_p), ("branch_norm", C.c_void_p),
                 ("in_taps", C.c_int), ("in_conv1", C.c_void_p), ("in_conv2", C.c_void_p), ("q_rank", C.c_int), ("head_gate", C.c_int),
-                ("dq_norm", C.c_void_p), ("w_uq", C.c_void_p), ("act_coef", C.c_void_p), ("act_limit", C.c_float), ("act_slope", C.c_float)]
+                ("dq_norm", C.c_void_p), ("w_uq", C.c_void_p), ("act_coef", C.c_void_p), ("act_limit", C.c_float), ("act_slope", C.c_float),
+                ("dist_slope", C.c_void_p), ("v_share", C.c_int), ("v_lambda", C.c_float), ("rot_pairs", C.c_int), ("rot_turns", C.c_void_p),
+                ("rot_amp", C.c_float), ("logit_bias", C.c_void_p)]
 
 
 class HybridBatch(C.Structure):
@@ -100,7 +102,7 @@ class HybridBatch(C.Structure):
 MIXER_ATTN_CHUNKED, MIXER_GLA, MIXER_LATENT, MIXER_ATTN_SCORED, MIXER_DELTA, MIXER_MLSTM, MIXER_SSD, MIXER_LINEAR, MIXER_MINGRU = 1, 2, 3, 4, 5, 6, 7, 8, 9
 ATTN_SOFTMAX, ATTN_SIGMOID = 0, 1
 MLP_NONE, MLP_MOE, MLP_DENSE = 0, 1, 2
-NORM_RMS_POST, NORM_DYT_PRE_POST, NORM_LN_PARALLEL, NORM_LN_PRE, NORM_RMS_SUM = 0, 1, 2, 3, 4
+NORM_RMS_POST, NORM_DYT_PRE_POST, NORM_LN_PARALLEL, NORM_LN_PRE, NORM_RMS_SUM, NORM_LN_POST = 0, 1, 2, 3, 4, 5
 ROUTE_SIGMOID, ROUTE_SOFTMAX = 0, 1
 ACT_RELU2, ACT_SILU, ACT_GELU_TANH, ACT_RELU, ACT_POLYNORM, ACT_CLAMP_GLU = 0, 1, 2, 3, 4, 5
 (PLAN_MIXED_IDS, PLAN_MIXED_STARTS, PLAN_MIXED_POS0, PLAN_MIXED_SLOTS, PLAN_MIXED_REQUESTS, PLAN_MIXED_BLOCK_TABLE,

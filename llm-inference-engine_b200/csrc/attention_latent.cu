@@ -8,13 +8,14 @@
 // per-head products are grouped GEMMs over the heads (rows grouped head by head: [heads, t_pad, *], t_pad a whole number of row tiles).
 // The same form serves prompt portions and single decoded tokens, so a position's logits do not depend on how its prompt was cut.
 //   * latent_prep_kernel: splits the fused projection: qn (un-rotated query part) regrouped by head, qr rotated, and -- for a layer with a
-//     cache of its own -- the latent row normed (fp32) and the key part rotated, appended to the pool.  Angles are formed in fp64.
+//     cache of its own -- the latent row normed (fp32) and the key part rotated, appended to the pool.  Angles are formed in fp64; the
+//     rotating pairs are (i, i + rot_dims/2) or neighbours (2i, 2i+1), their frequencies powers of a base or a table of turns per position.
 //   * latent_attn_kernel: one CTA per (token, head): sliding window (i sees j with 0 <= i - j < window), softmax in fp32 with a per-head
 //     sink logit in the denominator, weighted sum of the latent rows.
 //   * latent_attn_mma_kernel: the tensor-core form for 16-bit engines: one CTA per tile of <= 64 query rows that share their keys (64
 //     consecutive tokens of one sequence x one head), key tiles of one page through a cp.async ring, the value operand read from the
 //     key tile's own first columns.
-//   * latent_gate_kernel: back to token-major rows, times sigmoid(gate).
+//   * latent_gate_kernel: back to token-major rows, times sigmoid(gate) (or as they are).
 #include "hybrid_ops.cuh"
 
 #include <algorithm>
@@ -30,23 +31,35 @@ __global__ void __launch_bounds__(128)
 latent_prep_kernel(const T *__restrict__ proj, int ld, int q_col, int kv_col, T *__restrict__ qn, T *__restrict__ qr, T *__restrict__ pool,
                    const float *__restrict__ kv_norm, float eps, const int *__restrict__ tok_seq, const int *__restrict__ tok_pos,
                    const int *__restrict__ block_table, int mpps, int t_pad, int heads, int dim, int rot_dim, int kv_rank, int rot_dims,
-                   float rot_base, const T *__restrict__ kv_proj, int kv_ld) {
+                   float rot_base, const T *__restrict__ kv_proj, int kv_ld, LatentRotation rt) {
     extern __shared__ float cs[];  // cos[half] | sin[half]
     __shared__ float red[33];
     const int t = blockIdx.x, half = rot_dims / 2;
     const int pos = tok_pos[t];
     float *cosv = cs, *sinv = cs + half;
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
-        const double f = exp2(-2.0 * (double)i / (double)rot_dims * log2((double)rot_base));
-        double s, c;
-        sincos((double)pos * f, &s, &c);
-        cosv[i] = (float)c, sinv[i] = (float)s;
+        if (rt.turns) {  // the angle in turns, in fp64; only its fraction goes to fp32, so that a far position costs no bits
+            const double a = (double)pos * rt.turns[i];
+            float s, c;
+            sincospif(2.0f * (float)(a - rint(a)), &s, &c);
+            cosv[i] = c * rt.amp, sinv[i] = s * rt.amp;
+        } else {
+            const double f = exp2(-2.0 * (double)i / (double)rot_dims * log2((double)rot_base));
+            double s, c;
+            sincos((double)pos * f, &s, &c);
+            cosv[i] = (float)c * rt.amp, sinv[i] = (float)s * rt.amp;
+        }
     }
     __syncthreads();
     const T *row = proj + (size_t)t * ld;
     // r-th element of a rotated vector that starts at `v`
     auto rotated = [&](const T *v, int r) -> float {
         const float self = Elem<T>::to_f(v[r]);
+        if (rt.pairs) {
+            if (r >= rot_dims) return self;
+            const float other = Elem<T>::to_f(v[r ^ 1]), cv = cosv[r >> 1], sv = sinv[r >> 1];
+            return (r & 1) ? self * cv + other * sv : self * cv - other * sv;
+        }
         if (r < half) return self * cosv[r] - Elem<T>::to_f(v[r + half]) * sinv[r];
         if (r < rot_dims) return self * cosv[r - half] + Elem<T>::to_f(v[r - half]) * sinv[r - half];
         return self;
@@ -456,6 +469,21 @@ latent_gate_kernel(const T *__restrict__ ov, const T *__restrict__ gate_in, int 
                    int head_gate) {
     const int t = blockIdx.x;
     constexpr int V = Elem<T>::kVec;
+    if (!gate_in) {  // no gate
+        if (vdim % V == 0 && ((reinterpret_cast<size_t>(ov) | reinterpret_cast<size_t>(out)) & 15) == 0) {
+            const int pieces = vdim / V;
+            for (int idx = threadIdx.x; idx < heads * pieces; idx += blockDim.x) {
+                const int h = idx / pieces, c = (idx - h * pieces) * V;
+                st_v4(out + ((size_t)t * heads + h) * vdim + c, ld_v4(ov + ((size_t)h * t_pad + t) * vdim + c));
+            }
+            return;
+        }
+        for (int idx = threadIdx.x; idx < heads * vdim; idx += blockDim.x) {
+            const int h = idx / vdim, c = idx - h * vdim;
+            out[(size_t)t * heads * vdim + idx] = ov[((size_t)h * t_pad + t) * vdim + c];
+        }
+        return;
+    }
     if (head_gate) {  // one gate per head
         const T *gr = gate_in + (size_t)t * gate_ld;
         if (vdim % V == 0 && ((reinterpret_cast<size_t>(ov) | reinterpret_cast<size_t>(out)) & 15) == 0) {
@@ -549,13 +577,14 @@ int launch_rms_rows(int dtype, const void *in, int ld, const float *w, float eps
 
 int launch_latent_prep(int dtype, const void *proj, int ld, int q_col, int kv_col, void *qn, void *qr, void *pool, const float *kv_norm,
                        float eps, const int *tok_seq, const int *tok_pos, const int *block_table, int mpps, int tokens, int t_pad, int heads,
-                       int dim, int rot_dim, int kv_rank, int rot_dims, float rot_base, cudaStream_t st, const void *kv_proj, int kv_ld) {
+                       int dim, int rot_dim, int kv_rank, int rot_dims, float rot_base, cudaStream_t st, const void *kv_proj, int kv_ld,
+                       LatentRotation rot) {
     if (tokens == 0) return B200_OK;
     const size_t smem = (size_t)std::max(rot_dims, 2) * sizeof(float);
     B200_DISPATCH_DTYPE(dtype, {
         latent_prep_kernel<T><<<tokens, 128, smem, st>>>((const T *)proj, ld, q_col, kv_col, (T *)qn, (T *)qr, (T *)pool, kv_norm, eps, tok_seq,
                                                         tok_pos, block_table, mpps, t_pad, heads, dim, rot_dim, kv_rank, rot_dims, rot_base,
-                                                        (const T *)kv_proj, kv_ld);
+                                                        (const T *)kv_proj, kv_ld, rot);
     });
     return cuda_status("latent_prep launch");
 }

@@ -4,8 +4,11 @@
 //     rotation of the first rot_dims dimensions of every q and k head in INTERLEAVED pairs (2i, 2i+1) -- or in halves (i, i + rot_dims/2) --
 //     by the angle pos * base^(-2i/rot_dims), optionally with the long wavelengths slowed down; optionally every value head divided by its
 //     root mean square; q to a dense buffer, k and v to their pages;
-//   * scored_attn_kernel: every token of the batch against the keys of ITS sequence inside the window 0 <= i - j < window (0: all j <= i).
-//     score = cap(scale * q.k) - r1[h] * ln(1 + r2[h] * (i - j)) (cap(s) = c tanh(s / c) and the penalty are optional); weights either softmax over the visible keys or
+//     optionally the values are kept for later layers of the call, or take a share of the values an earlier layer kept;
+//   * scored_attn_kernel: every token of the batch against the keys of ITS sequence inside the window 0 <= i - j < window (0: all j <= i)
+//     and, optionally, inside its own block of `chunk` positions.
+//     score = cap(scale * q.k) - r1[h] * ln(1 + r2[h] * (i - j)) - slope[h] * (i - j) (cap(s) = c tanh(s / c) and both penalties are optional);
+//     weights either softmax over the visible keys (optionally with a sink logit per head in the denominator) or
 //     sigmoid(score + head_bias[h]) without any normalisation; optional sigmoid output gate; the result is scaled by out_scale and written
 //     with a row stride, so that several mixers fill one row of a shared output-projection input;
 //   * scored_attn_mma_kernel: the same for prompt portions on the tensor cores (16-bit engines, dim and vdim multiples of 16 up to 128).
@@ -26,7 +29,8 @@ __global__ void __launch_bounds__(256)
 scored_prep_kernel(const T *__restrict__ proj, int ld, int col0, const float *__restrict__ b_in, T *__restrict__ q_out, T *__restrict__ k_pool,
                    T *__restrict__ v_pool, const float *__restrict__ q_norm, const float *__restrict__ k_norm, float eps,
                    const int *__restrict__ tok_seq, const int *__restrict__ tok_pos, const int *__restrict__ block_table, int mpps, int heads,
-                   int kv_heads, int dim, int vdim, int rot_dims, float rot_base, ScoredPrepOptions opt) {
+                   int kv_heads, int dim, int vdim, int rot_dims, float rot_base, ScoredPrepOptions opt, T *__restrict__ v_keep,
+                   const T *__restrict__ v_mix, float lambda) {
     extern __shared__ float rot[];  // cos [rot_dims/2] | sin [rot_dims/2]
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
     const int pos = tok_pos[t], half = rot_dims / 2;
@@ -98,7 +102,9 @@ scored_prep_kernel(const T *__restrict__ proj, int ld, int col0, const float *__
     }
     for (int c = threadIdx.x; c < kv_heads * vdim; c += blockDim.x) {
         const int g = c / vdim, cc = c - g * vdim;
-        const float v = Elem<T>::to_f(row[vsrc + c]) + (bias ? bias[vsrc + c] : 0.0f);
+        float v = Elem<T>::to_f(row[vsrc + c]) + (bias ? bias[vsrc + c] : 0.0f);
+        if (v_keep) v_keep[(size_t)t * kv_heads * vdim + c] = Elem<T>::from_f(v);
+        if (v_mix) v = (1.0f - lambda) * v + lambda * Elem<T>::to_f(v_mix[(size_t)t * kv_heads * vdim + c]);
         v_pool[(((size_t)page * kv_heads + g) * kPageS + off) * vdim + cc] = Elem<T>::from_f(v);
     }
 }
@@ -112,6 +118,12 @@ __device__ __forceinline__ float tanh_fast(float z) {
     return copysignf(1.0f - __fdividef(2.0f, e + 1.0f), z);
 }
 
+// the first key position `pos` sees: inside the window (0: none) and, chunk > 0, inside its own block of that many positions
+__device__ __forceinline__ int first_key(int pos, int window, int chunk) {
+    const int w = window > 0 ? max(0, pos - window + 1) : 0;
+    return chunk > 0 ? max(w, pos - pos % chunk) : w;
+}
+
 // One CTA per (token, query head).  Shared memory: q[dim] | weights[keys] | partial[key groups][vdim] | red[33].
 template <typename T>
 __global__ void __launch_bounds__(512)
@@ -119,12 +131,12 @@ scored_attn_kernel(const T *__restrict__ q, const T *__restrict__ k_pool, const 
                    const float *__restrict__ dist_r1, const float *__restrict__ dist_r2, const T *__restrict__ gate_in, int gate_ld,
                    T *__restrict__ out, int out_ld, float out_scale, const int *__restrict__ tok_seq, const int *__restrict__ tok_pos,
                    const int *__restrict__ block_table, int mpps, int heads, int kv_heads, int dim, int vdim, float scale, int window,
-                   int sigmoid, int max_keys, int part_floats, const int *__restrict__ tok_list, float softcap) {
+                   int sigmoid, int max_keys, int part_floats, const int *__restrict__ tok_list, ScoredOptions opt) {
     extern __shared__ float sm[];
     const int t = tok_list ? tok_list[blockIdx.x] : blockIdx.x, h = blockIdx.y;
     const int g = h / (heads / kv_heads);
     const int pos = tok_pos[t];
-    const int first = window > 0 ? max(0, pos - window + 1) : 0;
+    const int first = first_key(pos, window, opt.chunk);
     const int nkeys = pos - first + 1;
     float *qs = sm;
     float *sc = qs + dim;
@@ -134,11 +146,13 @@ scored_attn_kernel(const T *__restrict__ q, const T *__restrict__ k_pool, const 
     for (int c = threadIdx.x; c < dim; c += blockDim.x) qs[c] = Elem<T>::to_f(q[((size_t)t * heads + h) * dim + c]);
     __syncthreads();
     const float r1 = dist_r1 ? dist_r1[h] : 0.0f, r2 = dist_r2 ? dist_r2[h] : 0.0f, hb = head_bias ? head_bias[h] : 0.0f;
+    const float softcap = opt.softcap, slope = opt.slope ? opt.slope[h] : 0.0f;
     constexpr int V = Elem<T>::kVec;
     const bool kvec = dim % V == 0, vvec = vdim % V == 0;
 
     // ---- scores: four adjacent lanes share a key row
-    float mx = -INFINITY;
+    const bool sunk = !sigmoid && opt.sink;
+    float mx = sunk ? opt.sink[h] : -INFINITY;
     {
         const int sub = threadIdx.x & 3, kslot = threadIdx.x >> 2, nslots = blockDim.x >> 2, pieces = dim / V;
         for (int j0 = 0; j0 < nkeys; j0 += nslots) {  // warp-uniform trip count: the shuffles below take every lane
@@ -164,6 +178,7 @@ scored_attn_kernel(const T *__restrict__ q, const T *__restrict__ k_pool, const 
             acc *= scale;
             if (softcap > 0.0f) acc = softcap * tanhf(acc / softcap);
             if (dist_r1) acc -= r1 * log1pf(r2 * (float)(pos - p));
+            acc = fmaf(-slope, (float)(pos - p), acc);
             if (sigmoid) acc = sigmoid_f(acc + hb);
             if (j < nkeys) {
                 if (sub == 0) sc[j] = acc;
@@ -180,7 +195,9 @@ scored_attn_kernel(const T *__restrict__ q, const T *__restrict__ k_pool, const 
             sc[j] = e;
             sum += e;
         }
-        inv = 1.0f / block_sum(sum, red);  // (its barriers also publish sc[])
+        sum = block_sum(sum, red);  // (its barriers also publish sc[])
+        if (sunk) sum += expf(opt.sink[h] - mx);  // the sink: a logit with no key and no value, counted once
+        inv = 1.0f / sum;
     } else {
         __syncthreads();
     }
@@ -304,7 +321,7 @@ __global__ void __launch_bounds__(128)
 scored_attn_mma_kernel(const T *__restrict__ q, const T *__restrict__ k_pool, const T *__restrict__ v_pool, const float *__restrict__ head_bias,
                        const float *__restrict__ dist_r1, const float *__restrict__ dist_r2, const T *__restrict__ gate_in, int gate_ld,
                        T *__restrict__ out, int out_ld, float out_scale, const int4 *__restrict__ tiles, const int *__restrict__ block_table,
-                       int mpps, int heads, int kv_heads, float scale, int window, int pen_len, float softcap) {
+                       int mpps, int heads, int kv_heads, float scale, int window, int pen_len, ScoredOptions opt) {
     extern __shared__ __align__(16) unsigned char smraw[];
     T *qs = reinterpret_cast<T *>(smraw);       // [64][DK]
     T *ks = qs + kTileQS * DK;                  // [2][64][DK]
@@ -319,7 +336,7 @@ scored_attn_mma_kernel(const T *__restrict__ q, const T *__restrict__ k_pool, co
     constexpr float kLog2e = 1.4426950408889634f;
 
     const int last = pos0 + nrows - 1;
-    const int first = window > 0 ? max(0, pos0 - window + 1) : 0;
+    const int first = first_key(pos0, window, opt.chunk);
     const int tile_lo = first / kPageS, tile_hi = last / kPageS;
 
     auto load_kv = [&](int kt, int stage) {
@@ -358,14 +375,20 @@ scored_attn_mma_kernel(const T *__restrict__ q, const T *__restrict__ k_pool, co
         ldsm4(qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], qs + swzs<DK>(warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, kk * 16 + (lane >> 4) * 8));
 
     // a capped score: cap * tanh(scale * s / cap), in the softmax form times log2(e)
+    const float softcap = opt.softcap;
     const bool capped = softcap > 0.0f;
     const float sl2 = capped ? scale / softcap : (SIG ? scale : scale * kLog2e), cap2 = SIG ? softcap : softcap * kLog2e;
     auto scaled = [&](float sv) { return capped ? cap2 * tanh_fast(sv * sl2) : sv * sl2; };
     const float hb = (SIG && head_bias) ? head_bias[h] : 0.0f;
     const bool has_pen = !SIG && dist_r1 != nullptr;
     const int p_a = pos0 + warp * 16 + gid, p_b = p_a + 8;  // rows gid and gid + 8 of this warp's 16
-    const int lo_a = window > 0 ? p_a - window + 1 : 0, lo_b = window > 0 ? p_b - window + 1 : 0;
+    const int lo_a = first_key(p_a, window, opt.chunk), lo_b = first_key(p_b, window, opt.chunk);
+    const float slope = opt.slope ? opt.slope[h] * (SIG ? 1.0f : kLog2e) : 0.0f;
     float m_a = -1e30f, m_b = -1e30f, l_a = 0.0f, l_b = 0.0f;
+    if (!SIG && opt.sink) {  // the sink is the initial running state: a key with that logit and a zero value
+        m_a = m_b = opt.sink[h] * kLog2e;
+        l_a = l_b = tig == 0 ? 1.0f : 0.0f;  // (the sum is kept per lane and joined at the end)
+    }
     float o[DV / 8][4];
 #pragma unroll
     for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f;
@@ -398,8 +421,8 @@ scored_attn_mma_kernel(const T *__restrict__ q, const T *__restrict__ k_pool, co
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int key = kt * kPageS + j * 8 + tig * 2 + e;
-                    w[e] = (key <= p_a && key >= lo_a) ? sigmoid_fast(scaled(s[j][e]) + hb) : 0.0f;
-                    w[2 + e] = (key <= p_b && key >= lo_b) ? sigmoid_fast(scaled(s[j][2 + e]) + hb) : 0.0f;
+                    w[e] = (key <= p_a && key >= lo_a) ? sigmoid_fast(fmaf(-slope, (float)(p_a - key), scaled(s[j][e])) + hb) : 0.0f;
+                    w[2 + e] = (key <= p_b && key >= lo_b) ? sigmoid_fast(fmaf(-slope, (float)(p_b - key), scaled(s[j][2 + e])) + hb) : 0.0f;
                 }
                 pf[j >> 1][(j & 1) * 2] = pack2s<T>(w[0], w[1]);
                 pf[j >> 1][(j & 1) * 2 + 1] = pack2s<T>(w[2], w[3]);
@@ -412,8 +435,8 @@ scored_attn_mma_kernel(const T *__restrict__ q, const T *__restrict__ k_pool, co
                 for (int e = 0; e < 2; ++e) {
                     const int key = kt * kPageS + j * 8 + tig * 2 + e;
                     const bool va = key <= p_a && key >= lo_a, vb = key <= p_b && key >= lo_b;
-                    s[j][e] = va ? scaled(s[j][e]) - (has_pen ? pen[p_a - key] : 0.0f) : -INFINITY;
-                    s[j][2 + e] = vb ? scaled(s[j][2 + e]) - (has_pen ? pen[p_b - key] : 0.0f) : -INFINITY;
+                    s[j][e] = va ? fmaf(-slope, (float)(p_a - key), scaled(s[j][e])) - (has_pen ? pen[p_a - key] : 0.0f) : -INFINITY;
+                    s[j][2 + e] = vb ? fmaf(-slope, (float)(p_b - key), scaled(s[j][2 + e])) - (has_pen ? pen[p_b - key] : 0.0f) : -INFINITY;
                     mx_a = fmaxf(mx_a, s[j][e]);
                     mx_b = fmaxf(mx_b, s[j][2 + e]);
                 }
@@ -492,27 +515,27 @@ template <typename T, int DK, int DV>
 static int launch_scored_mma_t(const void *q, const void *k_pool, const void *v_pool, const float *head_bias, const float *r1, const float *r2,
                                const void *gate_in, int gate_ld, void *out, int out_ld, float out_scale, const int *tiles, int n_tiles,
                                const int *block_table, int mpps, int heads, int kv_heads, float scale, int window, int sigmoid, cudaStream_t st,
-                               float softcap) {
+                               ScoredOptions opt) {
     const int pen_len = (!sigmoid && r1) ? window + kTileQS : 0;
     const size_t smem = (size_t)(kTileQS + 2 * kPageS) * DK * sizeof(T) + (size_t)2 * kPageS * DV * sizeof(T) + (size_t)pen_len * sizeof(float);
     auto kern = sigmoid ? scored_attn_mma_kernel<T, DK, DV, 1> : scored_attn_mma_kernel<T, DK, DV, 0>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     kern<<<dim3(n_tiles, heads), 128, smem, st>>>((const T *)q, (const T *)k_pool, (const T *)v_pool, head_bias, r1, r2, (const T *)gate_in, gate_ld,
                                                   (T *)out, out_ld, out_scale, (const int4 *)tiles, block_table, mpps, heads, kv_heads, scale, window,
-                                                  pen_len, softcap);
+                                                  pen_len, opt);
     return cuda_status("scored_attention (tensor core) launch");
 }
 
 int launch_scored_attention_tiles(int dtype, const void *q, const void *k_pool, const void *v_pool, const float *head_bias, const float *dist_r1,
                                   const float *dist_r2, const void *gate_in, int gate_ld, void *out, int out_ld, float out_scale,
                                   const int *tiles, int n_tiles, const int *block_table, int mpps, int heads, int kv_heads, int dim, int vdim,
-                                  float scale, int window, int sigmoid, cudaStream_t st, float softcap) {
+                                  float scale, int window, int sigmoid, cudaStream_t st, ScoredOptions opt) {
     if (n_tiles == 0) return B200_OK;
     if (!scored_attention_tiles_supported(dtype, dim, vdim, gate_ld, out_ld, window, dist_r1 != nullptr)) {
         set_error("scored_attention tiles: 16-bit dtypes, dim and vdim of 32 / 64 / 128, a penalty only with a window");
         return B200_ERR_UNSUPPORTED;
     }
-#define B200_SCORED_ARGS q, k_pool, v_pool, head_bias, dist_r1, dist_r2, gate_in, gate_ld, out, out_ld, out_scale, tiles, n_tiles, block_table, mpps, heads, kv_heads, scale, window, sigmoid, st, softcap
+#define B200_SCORED_ARGS q, k_pool, v_pool, head_bias, dist_r1, dist_r2, gate_in, gate_ld, out, out_ld, out_scale, tiles, n_tiles, block_table, mpps, heads, kv_heads, scale, window, sigmoid, st, opt
 #define B200_SCORED_DV(TT, DK)                                                     \
     do {                                                                           \
         if (vdim == 32) return launch_scored_mma_t<TT, DK, 32>(B200_SCORED_ARGS);  \
@@ -535,12 +558,12 @@ int launch_scored_attention_tiles(int dtype, const void *q, const void *k_pool, 
 int launch_scored_prep(int dtype, const void *proj, int ld, int col0, const float *b_in, void *q_out, void *k_pool, void *v_pool,
                        const float *q_norm, const float *k_norm, float eps, const int *tok_seq, const int *tok_pos, const int *block_table,
                        int mpps, int tokens, int heads, int kv_heads, int dim, int vdim, int rot_dims, float rot_base, cudaStream_t st,
-                       ScoredPrepOptions opt) {
+                       ScoredPrepOptions opt, ValueShare share) {
     if (tokens == 0) return B200_OK;
     B200_DISPATCH_DTYPE(dtype, {
         scored_prep_kernel<T><<<tokens, 256, (size_t)std::max(rot_dims, 2) * sizeof(float), st>>>(
             (const T *)proj, ld, col0, b_in, (T *)q_out, (T *)k_pool, (T *)v_pool, q_norm, k_norm, eps, tok_seq, tok_pos, block_table, mpps, heads,
-            kv_heads, dim, vdim, rot_dims, rot_base, opt);
+            kv_heads, dim, vdim, rot_dims, rot_base, opt, (T *)share.v_keep, (const T *)share.v_mix, share.lambda);
     });
     return cuda_status("scored_prep launch");
 }
@@ -548,7 +571,7 @@ int launch_scored_prep(int dtype, const void *proj, int ld, int col0, const floa
 int launch_scored_attention(int dtype, const void *q, const void *k_pool, const void *v_pool, const float *head_bias, const float *dist_r1,
                             const float *dist_r2, const void *gate_in, int gate_ld, void *out, int out_ld, float out_scale, const int *tok_seq,
                             const int *tok_pos, const int *block_table, int mpps, int tokens, int heads, int kv_heads, int dim, int vdim,
-                            float scale, int window, int sigmoid, int max_keys, cudaStream_t st, const int *tok_list, float softcap) {
+                            float scale, int window, int sigmoid, int max_keys, cudaStream_t st, const int *tok_list, ScoredOptions opt) {
     if (tokens == 0) return B200_OK;
     const int threads = max_keys >= 512 ? 512 : (max_keys >= 256 ? 256 : 128);  // long contexts: more keys in flight per CTA
     const int ngroups = threads >= vdim ? threads / vdim : 1;
@@ -562,7 +585,7 @@ int launch_scored_attention(int dtype, const void *q, const void *k_pool, const 
         if (smem > 48 * 1024) cudaFuncSetAttribute(scored_attn_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         scored_attn_kernel<T><<<dim3(tokens, heads), threads, smem, st>>>(
             (const T *)q, (const T *)k_pool, (const T *)v_pool, head_bias, dist_r1, dist_r2, (const T *)gate_in, gate_ld, (T *)out, out_ld, out_scale,
-            tok_seq, tok_pos, block_table, mpps, heads, kv_heads, dim, vdim, scale, window, sigmoid, max_keys, (int)part, tok_list, softcap);
+            tok_seq, tok_pos, block_table, mpps, heads, kv_heads, dim, vdim, scale, window, sigmoid, max_keys, (int)part, tok_list, opt);
     });
     return cuda_status("scored_attention launch");
 }

@@ -16,6 +16,8 @@
 //   moe:              router + shared gate (fp32) -> route -> plan -> gather (weight on the input) -> grouped up (+act) -> grouped down
 //                     shared expert: b200_linear up -> act -> b200_linear down
 //                     combine (sum of the token's expert rows + gate * shared) + post-norm + residual add, one kernel
+// (B200_NORM_LN_POST: x += m * layernorm(mixer(x)) * g1, x += m * layernorm(ff(x)) * g2 runs in the same loop; so does the scored attention mixer:
+//   per-head q/k norm + values + pool append -> attention -> output projection)
 // Pre-norm layers on residual streams (B200_NORM_LN_PRE): per sublayer ONE kernel rewrites all streams from the sublayer's result (two
 // mixers side by side arrive as two projected rows, each RMS-normed over the width) and leaves the next sublayer's layer-normed input:
 //   input projection -> mixer (scored attention | delta rule | state-space | linear attention; a second mixer beside it) -> output
@@ -169,7 +171,8 @@ template <int N> __device__ __forceinline__ void load_vec(const float *__restric
 //   y[t, :]  = y_dense[t, :] + y_bias                                                  (a dense sublayer), or
 //            = sum_k w(t, k) * (pair_row[t, k] >= 0 ? y_rows[pair_row[t, k], :] : h_in[t, :]) + shared_gate[t] * y_shared[t, :]
 //              with w = pair_weight (NULL: 1) and shared_gate NULL: 1; a pair without a row is an identity expert;
-//   x[t, :] += ls * norm(y[t, :])    norm = RMS (post = g) or Dynamic Tanh (post packed);   has_y == 0: x stays as it is;
+//   x[t, :] += ls * norm(y[t, :])    norm = RMS (post = g), Dynamic Tanh (post packed) or layer norm (post = weight, result times
+//                                    branch_scale);   has_y == 0: x stays as it is;
 //   h_out[t, :] = T(pre ? dyt(x[t, :]; pre) : x[t, :]): what the next sublayer's projections read.
 // h_in and h_out may be the same buffer: an element is read by the thread that overwrites it, before it does.
 template <typename T, bool VEC>
@@ -178,7 +181,7 @@ sublayer_residual_kernel(float *__restrict__ x, const T *__restrict__ y_dense, c
                          const int *__restrict__ pair_row, const float *__restrict__ pair_weight, int top, const T *__restrict__ y_shared,
                          const float *__restrict__ shared_gate, const T *h_in, int norm, const float *__restrict__ post,
                          const float *__restrict__ ls, float eps, const float *__restrict__ pre, int width, float *__restrict__ trace, T *h_out,
-                         int has_y) {
+                         int has_y, float branch_scale) {
     extern __shared__ __align__(16) float ys[];  // [width]
     __shared__ float red[33];
     constexpr int V = Elem<T>::kVec;
@@ -217,8 +220,8 @@ sublayer_residual_kernel(float *__restrict__ x, const T *__restrict__ y_dense, c
             _Pragma("unroll") for (int i = 0; i < step; ++i) v[i] = fmaf(sg, f[i], v[i]);
         }
     };
-    const bool rms = has_y && norm == B200_NORM_RMS_POST;
-    float inv = 1.0f;
+    const bool layer_norm = norm == B200_NORM_LN_POST, rms = has_y && (norm == B200_NORM_RMS_POST || layer_norm);
+    float inv = 1.0f, mean = 0.0f;
     if (rms) {  // the mean square needs the whole row first: the row waits in shared memory
         float ss = 0.0f;
         for (int c = threadIdx.x * step; c < width; c += blockDim.x * step) {
@@ -226,11 +229,18 @@ sublayer_residual_kernel(float *__restrict__ x, const T *__restrict__ y_dense, c
             result(c, v);
             _Pragma("unroll") for (int i = 0; i < step; ++i) {
                 ys[c + i] = v[i];
-                ss = fmaf(v[i], v[i], ss);
+                ss = layer_norm ? ss + v[i] : fmaf(v[i], v[i], ss);
             }
         }
         ss = block_sum(ss, red);
+        if (layer_norm) {  // the mean first, then the squared deviations from it
+            mean = ss / (float)width, ss = 0.0f;
+            for (int c = threadIdx.x * step; c < width; c += blockDim.x * step)
+                _Pragma("unroll") for (int i = 0; i < step; ++i) ss = fmaf(ys[c + i] - mean, ys[c + i] - mean, ss);
+            ss = block_sum(ss, red);
+        }
         inv = rsqrtf(ss / (float)width + eps);
+        if (layer_norm) inv *= branch_scale;
     }
     const float a_post = (has_y && !rms) ? post[2 * width] : 0.0f, a_pre = pre ? pre[2 * width] : 0.0f;
     for (int c = threadIdx.x * step; c < width; c += blockDim.x * step) {  // (RMS: a thread reads back the elements of ys it wrote)
@@ -249,7 +259,7 @@ sublayer_residual_kernel(float *__restrict__ x, const T *__restrict__ y_dense, c
             if (rms) {
                 if constexpr (vec) load_vec<V>(post + c, g);
                 else g[0] = post[c];
-                _Pragma("unroll") for (int i = 0; i < step; ++i) y[i] = ys[c + i] * inv * g[i];
+                _Pragma("unroll") for (int i = 0; i < step; ++i) y[i] = (ys[c + i] - mean) * inv * g[i];
             } else {  // Dynamic Tanh works element by element: one pass, nothing staged
                 result(c, y);
                 if constexpr (vec) dyt_apply_vec<V>(post, width, c, a_post, y);
@@ -534,8 +544,8 @@ gated_act_strided_kernel(const T *__restrict__ in, int in_ld, int gate_col, int 
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-final_ln_rows_kernel(const float *__restrict__ x, const int *__restrict__ rows, const float *__restrict__ p, float eps, float *__restrict__ out,
-                     T *__restrict__ out_t, int width) {
+final_ln_rows_kernel(const float *__restrict__ x, const int *__restrict__ rows, const float *__restrict__ p, int has_bias, float eps,
+                     float *__restrict__ out, T *__restrict__ out_t, int width) {
     __shared__ float red[33];
     const int i = blockIdx.x;
     const float *xr = x + (size_t)rows[i] * width;
@@ -546,7 +556,7 @@ final_ln_rows_kernel(const float *__restrict__ x, const int *__restrict__ rows, 
     for (int c = threadIdx.x; c < width; c += blockDim.x) sq = fmaf(xr[c] - mean, xr[c] - mean, sq);
     const float inv = rsqrtf(block_sum(sq, red) / (float)width + eps);
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
-        const float v = fmaf((xr[c] - mean) * inv, p[c], p[width + c]);
+        const float v = fmaf((xr[c] - mean) * inv, p[c], has_bias ? p[width + c] : 0.0f);
         out[(size_t)i * width + c] = v;
         if (out_t) out_t[(size_t)i * width + c] = Elem<T>::from_f(v);
     }
@@ -708,7 +718,7 @@ struct b200_hybrid {
     void *h = nullptr, *proj = nullptr, *mix = nullptr, *mix2 = nullptr, *y = nullptr, *xg = nullptr, *u = nullptr, *yrows = nullptr, *us = nullptr,
          *ys = nullptr, *lqn = nullptr, *lqr = nullptr, *lql = nullptr, *lol = nullptr, *lov = nullptr;
     float *lpart = nullptr, *rec = nullptr, *f32c = nullptr, *xs = nullptr;
-    void *cat = nullptr, *xc = nullptr;
+    void *cat = nullptr, *xc = nullptr, *vkeep = nullptr;
     double *turns = nullptr;                    // the sinusoidal position vector's frequencies, formed by the first call after set_scratch
     bool turns_ready = false;
     float *maps = nullptr;
@@ -720,7 +730,7 @@ struct b200_hybrid {
 namespace {
 
 struct Carve {
-    size_t x, f32a, f32b, xn, h, proj, mix, y, xg, u, yrows, us, ys, lqn, lqr, lql, lov, lpart, meta, moe_i, moe_f, rec, f32c, cat, xc, xs, turns, maps, total;
+    size_t x, f32a, f32b, xn, h, proj, mix, y, xg, u, yrows, us, ys, lqn, lqr, lql, lov, lpart, meta, moe_i, moe_f, rec, f32c, cat, xc, xs, turns, maps, vkeep, total;
 };
 
 // rows of the input projection and columns of the output projection that ONE mixer owns
@@ -755,12 +765,15 @@ int max_rows_of(const b200_hybrid_config_t &c, const b200_hybrid_layer_t &l) {
     return ((pairs + 127) / 128 + l.experts) * 128;  // the larger of the two row-tile sizes
 }
 
+int latent_gate_rows(const b200_hybrid_layer_t &l) { return l.head_gate == 2 ? 0 : (l.head_gate ? l.heads : l.heads * l.vdim); }
+
 int n_in_of(const b200_hybrid_layer_t &l) {
     if (l.norm == B200_NORM_LN_PARALLEL) return mixer_rows(l) + (l.side ? mixer_rows(*l.side) : 0) + (l.mlp == B200_MLP_DENSE ? 2 * l.expert_ff : 0);
     if (l.norm == B200_NORM_LN_PRE) return mixer_rows(l) + (l.side ? mixer_rows(*l.side) : 0);
+    if (l.mixer == B200_MIXER_ATTN_SCORED) return mixer_rows(l);
     if (l.mixer == B200_MIXER_ATTN_CHUNKED) return (2 * l.heads + l.kv_heads) * l.dim;
     if (l.mixer == B200_MIXER_LATENT)
-        return (l.q_rank > 0 ? l.q_rank : l.heads * (l.dim + l.rot_dim)) + (l.head_gate ? l.heads : l.heads * l.vdim) + (l.kv_from < 0 ? l.kv_rank + l.rot_dim : 0);
+        return (l.q_rank > 0 ? l.q_rank : l.heads * (l.dim + l.rot_dim)) + latent_gate_rows(l) + (l.kv_from < 0 ? l.kv_rank + l.rot_dim : 0);
     if (l.mixer == B200_MIXER_MINGRU) return 3 * l.vdim;
     return 2 * l.heads * l.dim + 2 * l.heads * l.vdim + l.decay_rank;
 }
@@ -769,7 +782,7 @@ Carve carve(const b200_hybrid *m) {
     const b200_hybrid_config_t &c = m->cfg;
     const size_t T = (size_t)c.max_tokens, es = c.dtype == B200_F32 ? 4 : 2;
     size_t n_in = 1, n_mix = 1, n_f32 = 1, rows = 0, ff = 1, sff = 1, experts = 1, top = 1, lqn = 0, lqr = 0, lql = 0, lov = 0, lheads = 0, lpart = 0;
-    size_t n_rec = 0, n_heads = 0, n_cat = 0, n_gru = 0;
+    size_t n_rec = 0, n_heads = 0, n_cat = 0, n_gru = 0, n_vkeep = 0;
     bool pre_norm = false;
     const size_t t_pad = (T + 127) / 128 * 128;  // rows per head of the latent mixer's grouped GEMMs
     for (int i = 0; i < c.num_layers; ++i) {
@@ -779,6 +792,8 @@ Carve carve(const b200_hybrid *m) {
         n_mix = std::max(n_mix, (size_t)l.heads * std::max(l.dim, l.vdim));
         n_f32 = std::max(n_f32, (size_t)l.heads * std::max(l.dim, l.vdim));
         n_mix = std::max(n_mix, (size_t)l.heads * l.vdim);
+        for (const b200_hybrid_layer_t *mx : {&l, l.side})
+            if (mx && mx->v_share == 1) n_vkeep = std::max(n_vkeep, (size_t)mx->kv_heads * mx->vdim);
         if (l.norm == B200_NORM_LN_PARALLEL || l.norm == B200_NORM_LN_PRE) {
             if (l.norm == B200_NORM_LN_PARALLEL) n_cat = std::max(n_cat, (size_t)cat_cols(l));
             else n_cat = std::max(n_cat, (size_t)l.heads * l.vdim), sff = std::max(sff, (size_t)3 * l.expert_ff), pre_norm = true;
@@ -841,7 +856,8 @@ Carve carve(const b200_hybrid *m) {
     k.xs = pre_norm ? align256(T * (size_t)std::max(c.streams, 1) * c.width * 4) : 0;
     k.turns = c.pos_base > 0.0f ? align256((size_t)(c.width + 1) / 2 * 8) : 0;
     k.maps = align256((T / kMingruChunk + (size_t)c.max_seqs) * kMingruMapRows * n_gru * 4);
-    k.total = k.maps + k.turns + k.xs + k.x + k.f32a + k.f32b + k.xn + k.h + k.proj + 2 * k.mix + k.y + k.xg + k.u + k.yrows + k.us + k.ys + k.lqn + k.lqr + 2 * k.lql +
+    k.vkeep = align256(T * n_vkeep * es);
+    k.total = k.vkeep + k.maps + k.turns + k.xs + k.x + k.f32a + k.f32b + k.xn + k.h + k.proj + 2 * k.mix + k.y + k.xg + k.u + k.yrows + k.us + k.ys + k.lqn + k.lqr + 2 * k.lql +
               k.lov + k.lpart + k.meta + k.moe_i + k.moe_f + k.rec + k.f32c + k.cat + k.xc;
     return k;
 }
@@ -901,6 +917,9 @@ static int check_scored_mixer(const b200_hybrid_layer_t *w) {
         B200_REQUIRE(w->window >= 0 && (w->attn_weight == B200_ATTN_SOFTMAX || w->attn_weight == B200_ATTN_SIGMOID), "hybrid_set_layer: bad window or weight kind");
         B200_REQUIRE((w->dist_r1 == nullptr) == (w->dist_r2 == nullptr), "hybrid_set_layer: the distance penalty needs both of its vectors");
         B200_REQUIRE((w->q_norm == nullptr) == (w->k_norm == nullptr), "hybrid_set_layer: q and k are normed together or not at all");
+        B200_REQUIRE(w->chunk >= 0 && (!w->sink || w->attn_weight == B200_ATTN_SOFTMAX), "hybrid_set_layer: negative chunk, or a sink without softmax weights");
+        B200_REQUIRE(w->v_share >= 0 && w->v_share <= 2 && (w->v_share == 0 || !w->v_norm), "hybrid_set_layer: shared values are those as projected: v_share %d does not go with v_norm",
+                     w->v_share);
     } else if (w->mixer == B200_MIXER_DELTA) {
         B200_REQUIRE(w->kv_heads > 0 && w->heads % w->kv_heads == 0, "hybrid_set_layer: heads %d not a multiple of kv_heads %d", w->heads, w->kv_heads);
         B200_REQUIRE(w->conv >= 1 && w->conv <= 64 && w->conv_w && w->a_log && w->out_norm && w->decay_rank >= 0, "hybrid_set_layer: delta-rule sizes / weights missing");
@@ -925,7 +944,7 @@ int b200_hybrid_set_layer(b200_hybrid_t *m, int layer, const b200_hybrid_layer_t
     B200_REQUIRE(m && w, "hybrid_set_layer: null argument");
     B200_REQUIRE(layer >= 0 && layer < m->cfg.num_layers, "hybrid_set_layer: layer %d outside [0, %d)", layer, m->cfg.num_layers);
     B200_REQUIRE(w->mixer >= B200_MIXER_ATTN_CHUNKED && w->mixer <= B200_MIXER_MINGRU, "hybrid_set_layer: unknown mixer kind %d", w->mixer);
-    B200_REQUIRE(w->norm >= B200_NORM_RMS_POST && w->norm <= B200_NORM_RMS_SUM, "hybrid_set_layer: unknown norm kind %d", w->norm);
+    B200_REQUIRE(w->norm >= B200_NORM_RMS_POST && w->norm <= B200_NORM_LN_POST, "hybrid_set_layer: unknown norm kind %d", w->norm);
     B200_REQUIRE(w->heads > 0 && w->dim > 0 && w->w_in && w->w_out, "hybrid_set_layer: mixer sizes / weights missing");
     if (w->norm == B200_NORM_LN_PARALLEL || w->norm == B200_NORM_LN_PRE) {
         // LN_PARALLEL: one norm, one input projection, one output projection; the mixers are of the kinds that read a shared projection
@@ -958,10 +977,10 @@ int b200_hybrid_set_layer(b200_hybrid_t *m, int layer, const b200_hybrid_layer_t
         m->scratch = nullptr;
         return B200_OK;
     }
-    B200_REQUIRE((w->mixer <= B200_MIXER_LATENT || w->mixer == B200_MIXER_MINGRU) && !w->side, "hybrid_set_layer: mixer kind %d needs the shared-norm or the pre-norm layer form", w->mixer);
+    B200_REQUIRE((w->mixer <= B200_MIXER_ATTN_SCORED || w->mixer == B200_MIXER_MINGRU) && !w->side, "hybrid_set_layer: mixer kind %d needs the shared-norm or the pre-norm layer form", w->mixer);
     B200_REQUIRE(m->cfg.loop_times == 0, "hybrid_set_layer: only shared-norm and pre-norm layers can be looped");
-    const bool sum = w->norm == B200_NORM_RMS_SUM;
-    if (w->norm == B200_NORM_RMS_POST || sum) B200_REQUIRE(w->norm1, "hybrid_set_layer: norm weight missing");
+    const bool sum = w->norm == B200_NORM_RMS_SUM, behind = w->norm == B200_NORM_RMS_POST || w->norm == B200_NORM_LN_POST;
+    if (behind || sum) B200_REQUIRE(w->norm1, "hybrid_set_layer: norm weight missing");
     else B200_REQUIRE(w->pre1 && w->post1, "hybrid_set_layer: norm parameters missing");
     if (sum) B200_REQUIRE(w->in_taps >= 0 && w->in_taps <= 64 && (w->in_taps == 0 || (w->in_conv1 && (w->mlp == B200_MLP_NONE || w->in_conv2))),
                           "hybrid_set_layer: input convolution of %d taps (at most 64) / its weights", w->in_taps);
@@ -980,12 +999,16 @@ int b200_hybrid_set_layer(b200_hybrid_t *m, int layer, const b200_hybrid_layer_t
         B200_REQUIRE(w->kv_from < layer, "hybrid_set_layer: layer %d cannot read the latent rows of layer %d", layer, w->kv_from);
         B200_REQUIRE(w->kv_from >= 0 || w->kv_norm, "hybrid_set_layer: latent row norm weight missing");
         B200_REQUIRE(w->q_rank >= 0 && (w->q_rank == 0 || (w->dq_norm && w->w_uq)), "hybrid_set_layer: the low-rank query's norm / up-projection missing");
+        B200_REQUIRE(w->head_gate >= 0 && w->head_gate <= 2 && (!w->rot_turns || w->rot_dims > 0), "hybrid_set_layer: bad gate form, or turns without rotating dimensions");
+    } else if (w->mixer == B200_MIXER_ATTN_SCORED) {
+        const int rc = check_scored_mixer(w);
+        if (rc != B200_OK) return rc;
     } else {
         B200_REQUIRE(w->vdim > 0 && w->decay_rank > 0 && w->tau > 0.0f && w->w_decay && w->out_norm, "hybrid_set_layer: gla sizes / weights missing");
     }
     B200_REQUIRE(w->mlp == B200_MLP_NONE || w->mlp == B200_MLP_MOE || w->mlp == B200_MLP_DENSE, "hybrid_set_layer: unknown feed-forward kind %d", w->mlp);
     if (w->mlp != B200_MLP_NONE) {
-        if (w->norm == B200_NORM_RMS_POST || sum) B200_REQUIRE(w->norm2, "hybrid_set_layer: feed-forward norm weight missing");
+        if (behind || sum) B200_REQUIRE(w->norm2, "hybrid_set_layer: feed-forward norm weight missing");
         else B200_REQUIRE(w->pre2 && w->post2, "hybrid_set_layer: feed-forward norm parameters missing");
         B200_REQUIRE(w->act >= B200_ACT_RELU2 && w->act <= B200_ACT_CLAMP_GLU, "hybrid_set_layer: unknown activation %d", w->act);
         if (w->act == B200_ACT_POLYNORM)
@@ -1068,6 +1091,7 @@ int b200_hybrid_set_scratch(b200_hybrid_t *m, void *ptr, size_t bytes) {
     m->xs = (float *)p, p += k.xs;
     m->turns = (double *)p, p += k.turns, m->turns_ready = false;
     m->maps = (float *)p, p += k.maps;
+    m->vkeep = p, p += k.vkeep;
     return B200_OK;
 }
 
@@ -1141,10 +1165,17 @@ int b200_hybrid_set_pools(b200_hybrid_t *m, void *kv_pool, int num_pages, void *
         place_mixer(l, es, num_pages, num_slots, kv, stt, &lp);
         if (l.side) place_mixer(*l.side, es, num_pages, num_slots, kv, stt, &lp.side);
         place_conv(l, m->cfg.width, num_slots, stt, lp.conv_off);
+        if (l.v_share == 2) {  // values of an earlier layer join this layer's: the last one before it that keeps its own, with equal sizes
+            int from = i - 1;
+            while (from >= 0 && m->layers[from].v_share != 1) --from;
+            B200_REQUIRE(from >= 0 && m->layers[from].kv_heads == l.kv_heads && m->layers[from].vdim == l.vdim,
+                         "hybrid_set_pools: layer %d mixes in an earlier layer's values, and none of equal sizes keeps its own", i);
+        }
         if (l.mixer == B200_MIXER_LATENT && l.kv_from >= 0) {  // the rows of an earlier layer, which must own them and rotate them alike
             const b200_hybrid_layer_t &o = m->layers[l.kv_from];
             B200_REQUIRE(o.mixer == B200_MIXER_LATENT && o.kv_from < 0 && o.kv_rank == l.kv_rank && o.rot_dim == l.rot_dim &&
-                             o.rot_dims == l.rot_dims && o.rot_base == l.rot_base,
+                             o.rot_dims == l.rot_dims && o.rot_base == l.rot_base && o.rot_pairs == l.rot_pairs && o.rot_turns == l.rot_turns &&
+                             o.rot_amp == l.rot_amp,
                          "hybrid_set_pools: layer %d cannot read the latent rows of layer %d (no cache of its own, or other sizes)", i, l.kv_from);
             lp.k_off = m->plan[l.kv_from].k_off;  // (latent layers are never looped: run == layer)
         }
@@ -1320,17 +1351,23 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
             ScoredPrepOptions opt;
             opt.rot_half = l.rot_half, opt.rot_factor = l.rot_factor, opt.rot_low = l.rot_low, opt.rot_high = l.rot_high, opt.rot_original = l.rot_original;
             opt.v_norm = l.v_norm;
+            ValueShare share;
+            if (l.v_share == 1) share.v_keep = m->vkeep;
+            if (l.v_share == 2) share.v_mix = m->vkeep, share.lambda = l.v_lambda;
+            ScoredOptions so;
+            so.softcap = l.softcap, so.slope = l.dist_slope, so.chunk = l.chunk, so.sink = l.sink;
             RUN(launch_scored_prep(dt, m->proj, n_in, col, l.b_in, m->mix, kp, vp, l.q_norm, l.k_norm, c.norm_eps, d_seq, d_pos, d_bt, mpps, NT, l.heads,
-                                   l.kv_heads, l.dim, l.vdim, l.rot_dims, l.rot_base, st, opt));
-            const int max_keys = l.window > 0 ? std::min(l.window, mpps * kPageH) : mpps * kPageH;
+                                   l.kv_heads, l.dim, l.vdim, l.rot_dims, l.rot_base, st, opt, share));
+            int max_keys = l.window > 0 ? std::min(l.window, mpps * kPageH) : mpps * kPageH;
+            if (l.chunk > 0) max_keys = std::min(max_keys, l.chunk);
             if (scored_attention_tiles_supported(dt, l.dim, l.vdim, n_in, out_ld, l.window, l.dist_r1 != nullptr)) {
                 RUN(launch_scored_attention_tiles(dt, m->mix, kp, vp, l.head_bias, l.dist_r1, l.dist_r2, gate, n_in, out, out_ld, out_scale, d_tiles, n_tiles,
-                                                  d_bt, mpps, l.heads, l.kv_heads, l.dim, l.vdim, l.scale, l.window, sig, st, l.softcap));
+                                                  d_bt, mpps, l.heads, l.kv_heads, l.dim, l.vdim, l.scale, l.window, sig, st, so));
                 RUN(launch_scored_attention(dt, m->mix, kp, vp, l.head_bias, l.dist_r1, l.dist_r2, gate, n_in, out, out_ld, out_scale, d_seq, d_pos, d_bt,
-                                            mpps, n_short, l.heads, l.kv_heads, l.dim, l.vdim, l.scale, l.window, sig, max_keys, st, d_short, l.softcap));
+                                            mpps, n_short, l.heads, l.kv_heads, l.dim, l.vdim, l.scale, l.window, sig, max_keys, st, d_short, so));
             } else {
                 RUN(launch_scored_attention(dt, m->mix, kp, vp, l.head_bias, l.dist_r1, l.dist_r2, gate, n_in, out, out_ld, out_scale, d_seq, d_pos, d_bt,
-                                            mpps, NT, l.heads, l.kv_heads, l.dim, l.vdim, l.scale, l.window, sig, max_keys, st, nullptr, l.softcap));
+                                            mpps, NT, l.heads, l.kv_heads, l.dim, l.vdim, l.scale, l.window, sig, max_keys, st, nullptr, so));
             }
         } else if (l.mixer == B200_MIXER_DELTA) {
             float *conv_state = (float *)(m->state_pool + mp.aux_off);
@@ -1521,7 +1558,8 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
             auto kern = vec ? sublayer_residual_kernel<T, true> : sublayer_residual_kernel<T, false>;
             kern<<<NT, 256, (size_t)width * sizeof(float), st>>>(m->x, (const T *)y_dense, y_bias, (const T *)y_rows, pair_row, pair_weight, top,
                                                                 (const T *)y_shared, gate, (const T *)m->h, norm, post, ls, c.norm_eps, pre, width, trace,
-                                                                (pre || !f32) ? (T *)m->h : nullptr, has_y ? 1 : 0);
+                                                                (pre || !f32) ? (T *)m->h : nullptr, has_y ? 1 : 0,
+                                                                c.branch_scale != 0.0f ? c.branch_scale : 1.0f);
         });
         return cuda_status("sublayer_residual launch");
     };
@@ -1545,7 +1583,7 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
         }
         const b200_hybrid_layer_t &l = m->layers[li];
         const LayerPlan &lp = m->plan[li];
-        const bool dyt = l.norm == B200_NORM_DYT_PRE_POST;
+        const bool dyt = l.norm == B200_NORM_DYT_PRE_POST, ln_post = l.norm == B200_NORM_LN_POST;
         float *trace = (layer_trace && l.mlp == B200_MLP_NONE) ? layer_trace + (size_t)li * NT * width : nullptr;
         if (dyt && !h_normed) RUN(residual(false, nullptr, nullptr, nullptr, nullptr, nullptr, 0, nullptr, nullptr, l.norm, nullptr, nullptr, l.pre1, nullptr));
         const void *h = dyt || sum_norm ? (const void *)m->h : cast_x();
@@ -1567,19 +1605,24 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
                                              d_bt, mpps, NT, l.heads, l.kv_heads, l.dim, l.scale, l.chunk, max_keys, st));
             }
             n_mixed = hd;
+        } else if (l.mixer == B200_MIXER_ATTN_SCORED) {
+            n_mixed = l.heads * l.vdim;
+            RUN(run_mixer(l, lp, lp.n_in, 0, m->mix2, n_mixed, 1.0f));
         } else if (l.mixer == B200_MIXER_LATENT) {
             const int nq = l.heads * (l.dim + l.rot_dim), hv = l.heads * l.vdim;
             const bool low_q = l.q_rank > 0;
             const int gate_col = low_q ? l.q_rank + (l.kv_from < 0 ? l.kv_rank + l.rot_dim : 0) : nq;
-            const char *gate = (const char *)m->proj + (size_t)gate_col * es;
+            const char *gate = l.head_gate == 2 ? nullptr : (const char *)m->proj + (size_t)gate_col * es;
+            LatentRotation rot;
+            rot.pairs = l.rot_pairs, rot.turns = l.rot_turns, rot.amp = l.rot_amp != 0.0f ? l.rot_amp : 1.0f;
             char *pool = m->kv_pool + lp.k_off;
             if (low_q) {  // the queries come through a normed low-rank row
                 RUN(launch_rms_rows(dt, m->proj, lp.n_in, l.dq_norm, c.norm_eps, m->mix2, NT, l.q_rank, st));
                 RUN(linear(m, m->mix2, l.w_uq, m->mix, NT, l.q_rank, nq, st));
             }
-            const int kv_col = l.kv_from >= 0 ? -1 : (low_q ? l.q_rank : nq + (l.head_gate ? l.heads : hv));
+            const int kv_col = l.kv_from >= 0 ? -1 : (low_q ? l.q_rank : nq + latent_gate_rows(l));
             RUN(launch_latent_prep(dt, low_q ? m->mix : m->proj, low_q ? nq : lp.n_in, 0, kv_col, m->lqn, m->lqr, pool, l.kv_norm, c.norm_eps, d_seq, d_pos,
-                                   d_bt, mpps, NT, t_pad, l.heads, l.dim, l.rot_dim, l.kv_rank, l.rot_dims, l.rot_base, st, low_q ? m->proj : nullptr, lp.n_in));
+                                   d_bt, mpps, NT, t_pad, l.heads, l.dim, l.rot_dim, l.kv_rank, l.rot_dims, l.rot_base, st, low_q ? m->proj : nullptr, lp.n_in, rot));
             // the per-head products: rows past the batch's tokens hold whatever the scratch held; a row of a product depends on its own
             // input row only and those rows are never read
             auto head_product = [&](const void *a, const void *w, void *out, int N, int K) -> int {
@@ -1625,6 +1668,8 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
         RUN(linear(m, m->mix2, l.w_out, m->y, NT, n_mixed, width, st));
         if (sum_norm) {
             RUN(sum_step(li, 0, m->y, nullptr, nullptr, nullptr, nullptr, trace));
+        } else if (ln_post) {
+            RUN(residual(true, m->y, nullptr, nullptr, nullptr, nullptr, 0, nullptr, nullptr, l.norm, l.norm1, nullptr, nullptr, trace));
         } else if (dyt) {
             const float *pre = next_pre(li, 0);
             RUN(residual(true, m->y, nullptr, nullptr, nullptr, nullptr, 0, nullptr, nullptr, l.norm, l.post1, l.ls1, pre, trace));
@@ -1678,7 +1723,7 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
             rc = dyt || sum_norm ? launch_proj_f32(dt, m->h, width, dt, l.w_router, nullptr, m->f32a, outputs, NT, outputs, width, st)
                      : launch_proj_f32(B200_F32, m->x, width, dt, l.w_router, nullptr, m->f32a, outputs, NT, outputs, width, st);
         if (rc != B200_OK) return rc;
-        if (softmax) RUN(launch_moe_route_softmax(m->f32a, outputs, l.route_bias, sel_expert, sel_weight, NT, outputs, l.top, st));
+        if (softmax) RUN(launch_moe_route_softmax(m->f32a, outputs, l.route_bias, sel_expert, sel_weight, NT, outputs, l.top, st, l.logit_bias));
         else RUN(launch_moe_route_sigmoid(m->f32a, outputs, sel_expert, sel_weight, l.shared_ff > 0 ? shared_gate : nullptr, NT, l.experts, l.top, st));
         RUN(launch_moe_plan(sel_expert, sel_weight, row_token, row_weight, tile_expert, pair_row, n_live, NT, l.experts, l.top, tile, st));
         if (softmax || sum_norm)  // sigmoid scores weigh the experts' inputs: the fp32 residual row, or the convolved row the router read
@@ -1721,7 +1766,8 @@ int b200_hybrid_forward(b200_hybrid_t *m, const b200_hybrid_batch_t *b, float *l
     if (W > 0) {
         // the wanted rows only: final norm (fp32 and, for 16-bit engines, a 16-bit copy in h), then the LM head with fp32 logits
         B200_DISPATCH_DTYPE(dt, {
-            if (c.final_norm == B200_NORM_LN_PARALLEL || c.final_norm == B200_NORM_LN_PRE) final_ln_rows_kernel<T><<<W, 256, 0, st>>>(m->x, d_want, m->final_norm, c.norm_eps, m->xn, f32 ? nullptr : (T *)m->h, width);
+            if (c.final_norm == B200_NORM_LN_PARALLEL || c.final_norm == B200_NORM_LN_PRE || c.final_norm == B200_NORM_LN_POST)
+                final_ln_rows_kernel<T><<<W, 256, 0, st>>>(m->x, d_want, m->final_norm, c.final_norm != B200_NORM_LN_POST, c.norm_eps, m->xn, f32 ? nullptr : (T *)m->h, width);
             else if (c.final_norm == B200_NORM_DYT_PRE_POST) final_dyt_rows_kernel<T><<<W, 256, 0, st>>>(m->x, d_want, m->final_norm, m->xn, f32 ? nullptr : (T *)m->h, width);
             else final_norm_rows_kernel<T><<<W, 256, 0, st>>>(m->x, d_want, m->final_norm, c.norm_eps, m->xn, f32 ? nullptr : (T *)m->h, width);
         });

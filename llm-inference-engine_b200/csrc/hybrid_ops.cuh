@@ -17,11 +17,16 @@ int launch_chunked_attention_tiles(int dtype, const void *q, const void *k_pool,
                                    int gate_ld, void *out, const int *tiles, int n_tiles, const int *block_table, int mpps, int heads,
                                    int kv_heads, int dim, float scale, int chunk, cudaStream_t st);
 
-// attention_latent.cu (layouts in the file's header): proj [tokens, ld] holds q at column q_col and, when kv_col >= 0, the down-projection
+// attention_latent.cu
+// other rotations than pairs (i, i + rot_dims/2) by pos * rot_base^(-2i/rot_dims): pairs: (2i, 2i+1); turns: DEVICE [rot_dims/2] turns per
+// position of every pair instead of the powers of rot_base; amp multiplies cosine and sine
+struct LatentRotation { int pairs = 0; const double *turns = nullptr; float amp = 1.0f; };
+// (layouts in the file's header): proj [tokens, ld] holds q at column q_col and, when kv_col >= 0, the down-projection
 // (in kv_proj [tokens, kv_ld] instead, if given)
 int launch_latent_prep(int dtype, const void *proj, int ld, int q_col, int kv_col, void *qn, void *qr, void *pool, const float *kv_norm,
                        float eps, const int *tok_seq, const int *tok_pos, const int *block_table, int mpps, int tokens, int t_pad, int heads,
-                       int dim, int rot_dim, int kv_rank, int rot_dims, float rot_base, cudaStream_t st, const void *kv_proj = nullptr, int kv_ld = 0);
+                       int dim, int rot_dim, int kv_rank, int rot_dims, float rot_base, cudaStream_t st, const void *kv_proj = nullptr, int kv_ld = 0,
+                       LatentRotation rot = LatentRotation());
 int launch_latent_attention(int dtype, const void *ql, const void *qr, const void *pool, const float *sink, void *ol, const int *tok_seq,
                             const int *tok_pos, const int *block_table, int mpps, int tokens, int t_pad, int heads, int kv_rank, int rot_dim,
                             float scale, int window, int max_keys, cudaStream_t st, const int *tok_list = nullptr);
@@ -32,7 +37,7 @@ bool latent_attention_tiles_supported(int dtype, int kv_rank, int rot_dim);
 int launch_latent_attention_tiles(int dtype, const void *ql, const void *qr, const void *pool, const float *sink, void *ol, const int *tiles,
                                   int n_tiles, const int *block_table, int mpps, int t_pad, int heads, int kv_rank, int rot_dim, float scale,
                                   int window, int by_head, float *part, int part_tiles, cudaStream_t st);
-// head_gate: gate_in holds ONE number per head instead of one per value channel
+// gate_in NULL: no gate (the rows only go back to token-major order); head_gate: gate_in holds ONE number per head instead of one per value channel
 int launch_latent_gate(int dtype, const void *ov, const void *gate_in, int gate_ld, void *out, int tokens, int t_pad, int heads, int vdim,
                        cudaStream_t st, int head_gate = 0);
 // out [tokens, cols] = rmsnorm(in [tokens, ld] from its column 0 on) * w
@@ -43,20 +48,26 @@ int launch_rms_rows(int dtype, const void *in, int ld, const float *w, float eps
 // options of the prep step: rot_half: rotating pairs (i, i + rot_dims/2) instead of (2i, 2i+1); rot_factor > 0: long wavelengths are slowed
 // down (b200_hybrid_layer_t); v_norm: value heads are cached divided by their root mean square
 struct ScoredPrepOptions { int rot_half = 0; float rot_factor = 0.0f, rot_low = 0.0f, rot_high = 0.0f, rot_original = 0.0f; int v_norm = 0; };
+// v_keep [tokens, kv_heads*vdim]: receives the values as projected; v_mix: values of the same shape that join this layer's, v <- (1 - lambda) v +
+// lambda * v_mix, before they are cached
+struct ValueShare { void *v_keep = nullptr; const void *v_mix = nullptr; float lambda = 0.0f; };
+// what else enters a score or a softmax: slope [heads]: score -= slope * distance; chunk > 0: i sees j in its own block of this many positions
+// only; sink [heads] (softmax weights): a logit without a value in the denominator
+struct ScoredOptions { float softcap = 0.0f; const float *slope = nullptr; int chunk = 0; const float *sink = nullptr; };
 int launch_scored_prep(int dtype, const void *proj, int ld, int col0, const float *b_in, void *q_out, void *k_pool, void *v_pool,
                        const float *q_norm, const float *k_norm, float eps, const int *tok_seq, const int *tok_pos, const int *block_table,
                        int mpps, int tokens, int heads, int kv_heads, int dim, int vdim, int rot_dims, float rot_base, cudaStream_t st,
-                       ScoredPrepOptions opt = ScoredPrepOptions());
+                       ScoredPrepOptions opt = ScoredPrepOptions(), ValueShare share = ValueShare());
 int launch_scored_attention(int dtype, const void *q, const void *k_pool, const void *v_pool, const float *head_bias, const float *dist_r1,
                             const float *dist_r2, const void *gate_in, int gate_ld, void *out, int out_ld, float out_scale, const int *tok_seq,
                             const int *tok_pos, const int *block_table, int mpps, int tokens, int heads, int kv_heads, int dim, int vdim,
                             float scale, int window, int sigmoid, int max_keys, cudaStream_t st, const int *tok_list = nullptr,
-                            float softcap = 0.0f);
+                            ScoredOptions opt = ScoredOptions());
 bool scored_attention_tiles_supported(int dtype, int dim, int vdim, int gate_ld, int out_ld, int window, bool penalty);
 int launch_scored_attention_tiles(int dtype, const void *q, const void *k_pool, const void *v_pool, const float *head_bias, const float *dist_r1,
                                   const float *dist_r2, const void *gate_in, int gate_ld, void *out, int out_ld, float out_scale,
                                   const int *tiles, int n_tiles, const int *block_table, int mpps, int heads, int kv_heads, int dim, int vdim,
-                                  float scale, int window, int sigmoid, cudaStream_t st, float softcap = 0.0f);
+                                  float scale, int window, int sigmoid, cudaStream_t st, ScoredOptions opt = ScoredOptions());
 
 // recurrent.cu: column offsets of the fp32 row per token that the prep kernels write and the recurrences read.
 // launch_delta_prep scratch: lr (engine dtype) of tokens * (rank + gate_rank) elements + 256 bytes, za fp32 [tokens, heads*dim], zg fp32
@@ -143,9 +154,10 @@ int launch_gla_output(int dtype, const float *o, const float *w, float eps, cons
 // moe.cu
 int launch_moe_route_sigmoid(const float *logits, int ld, int *sel_expert, float *sel_weight, float *shared_gate, int tokens,
                              int experts, int top, cudaStream_t st);
-// scores = softmax over `outputs` router outputs; choice by score + bias (NULL: none); weights = chosen scores / (their sum + 1e-20)
+// scores = softmax over `outputs` router outputs (logits + logit_bias; NULL: none); choice by score + bias (NULL: by the logit itself); weights =
+// chosen scores / (their sum + 1e-20)
 int launch_moe_route_softmax(const float *logits, int ld, const float *bias, int *sel_expert, float *sel_weight, int tokens, int outputs,
-                             int top, cudaStream_t st);
+                             int top, cudaStream_t st, const float *logit_bias = nullptr);
 constexpr int kMoeTileM = 64;  // rows of one expert are padded to whole tiles of this many (128 when the tcgen05 grouped GEMM runs)
 // Groups the (token, choice) pairs by expert.  row_token / row_weight [max_rows]: token of every padded row (-1: padding) and its routing
 // weight; tile_expert [max_tiles]; pair_row [tokens*top]: the row each pair landed in (-1 for a choice >= experts: an identity expert);

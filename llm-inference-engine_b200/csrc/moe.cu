@@ -47,17 +47,19 @@ __global__ void moe_route_sigmoid_kernel(const float *__restrict__ logits, int l
     if (lane == 0 && shared_gate) shared_gate[t] = 1.0f / (1.0f + expf(-z[experts]));
 }
 
-// one warp per token; `outputs` router outputs (real experts first, then identity experts)
-__global__ void moe_route_softmax_kernel(const float *__restrict__ logits, int ld, const float *__restrict__ bias, int *__restrict__ sel_expert,
-                                         float *__restrict__ sel_weight, int tokens, int outputs, int top) {
+// one warp per token; `outputs` router outputs (real experts first, then identity experts).  Without a choice bias the choice is made on the
+// logits, which order the scores and do not underflow.
+__global__ void moe_route_softmax_kernel(const float *__restrict__ logits, int ld, const float *__restrict__ bias, const float *__restrict__ logit_bias,
+                                         int *__restrict__ sel_expert, float *__restrict__ sel_weight, int tokens, int outputs, int top) {
     const int t = blockIdx.x * (blockDim.x / 32) + threadIdx.x / 32, lane = threadIdx.x & 31;
     if (t >= tokens) return;
-    const float *z = logits + (size_t)t * ld;
+    const float *row = logits + (size_t)t * ld;
+    auto z = [&](int e) { return row[e] + (logit_bias ? logit_bias[e] : 0.0f); };
     float mx = -INFINITY;
-    for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, z[e]);
+    for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, z(e));
     mx = warp_max(mx);
     float den = 0.0f;
-    for (int e = lane; e < outputs; e += 32) den += expf(z[e] - mx);
+    for (int e = lane; e < outputs; e += 32) den += expf(z(e) - mx);
     den = warp_sum(den);
     const float inv = 1.0f / den;
     float chosen_sum = 0.0f;
@@ -67,8 +69,8 @@ __global__ void moe_route_softmax_kernel(const float *__restrict__ logits, int l
         for (int e = lane; e < outputs; e += 32) {
             bool taken = false;
             for (int p = 0; p < k; ++p) taken |= sel_expert[(size_t)t * top + p] == e;
-            const float sc = expf(z[e] - mx) * inv;
-            const float v = sc + (bias ? bias[e] : 0.0f);
+            const float ze = z(e), sc = expf(ze - mx) * inv;
+            const float v = bias ? sc + bias[e] : ze;
             if (!taken && (v > best || (v == best && e < bi))) best = v, bi = e, best_s = sc;
         }
         for (int o = 16; o > 0; o >>= 1) {
@@ -517,9 +519,9 @@ int launch_moe_route_sigmoid(const float *logits, int ld, int *sel_expert, float
 }
 
 int launch_moe_route_softmax(const float *logits, int ld, const float *bias, int *sel_expert, float *sel_weight, int tokens, int outputs,
-                             int top, cudaStream_t st) {
+                             int top, cudaStream_t st, const float *logit_bias) {
     if (tokens == 0) return B200_OK;
-    moe_route_softmax_kernel<<<(tokens + 3) / 4, 128, 0, st>>>(logits, ld, bias, sel_expert, sel_weight, tokens, outputs, top);
+    moe_route_softmax_kernel<<<(tokens + 3) / 4, 128, 0, st>>>(logits, ld, bias, logit_bias, sel_expert, sel_weight, tokens, outputs, top);
     return cuda_status("moe_route (softmax) launch");
 }
 

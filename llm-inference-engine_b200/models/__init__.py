@@ -26,7 +26,7 @@ def architectures():
 
 
 def _populate():
-    for sub in ("vasolix", "zefenex", "fedovik", "silonex", "zasapel", "llama"):
+    for sub in ("vasolix", "zefenex", "fedovik", "silonex", "zasapel", "pamulix", "llama"):
         importlib.import_module(f"{__name__}.{sub}")
 
 
