@@ -1277,6 +1277,41 @@ def zefenex_model(lb, sz):
     return model, 2.0 * lb.tokens * lat_active + lat_attn_flops, lat_w_bytes + lat_kv_bytes
 
 
+def vasolix_model(lb, sz):
+    """Four chunked-attention layers (values = keys, whole-projection norms, the window of `sz` as the chunk; 0: causal) with sigmoid-routed
+    experts: the Vasolix-shaped model of the numbers `sz`, with the FLOPs of its prefill and the bytes of its decode step."""
+    import torch
+
+    W, H, M, V, Tq, B, d, chunk = sz["width"], sz["heads"], sz["moe"], lb.vocab, lb.tokens, lb.batch, sz["dim"], sz["window"]
+    rnd, ones, Gk = lb.rnd, lb.ones, max(1, H // 4)
+    mixer = {"heads": H, "kv_heads": Gk, "dim": d, "vdim": d, "scale": d ** -0.5}
+    if chunk:
+        mixer["mask"] = {"size": chunk}
+    moe = {"kind": "moe", "expert": {"ff": M["ff"]}, "router": {"experts": M["experts"], "top": M["top"]}}
+    if M["shared"]:
+        moe["shared"] = {"ff": M["shared"]}
+    config = {"architecture": "Vasolix", "layers": [{"type": "attention", "mixer": mixer, "mlp": moe}] * 4, "norm": {"eps": 1e-6}, "vocab": V, "width": W}
+    t = {"embed": rnd(V, W, std=1.0), "head": rnd(V, W), "final.norm": ones(W)}
+    for i in range(4):
+        p = f"l{i}."
+        t[p + "norm1"], t[p + "norm2"] = ones(W), ones(W)
+        t.update({p + "mix.q": rnd(H * d, W), p + "mix.k": rnd(Gk * d, W), p + "mix.g": rnd(H * d, W), p + "mix.o": rnd(W, H * d),
+                  p + "mix.q.norm": ones(H * d), p + "mix.k.norm": ones(Gk * d), p + "mix.sink": torch.zeros(H, dtype=torch.bfloat16)})
+        t[p + "mlp.router"] = rnd(M["experts"], W)
+        up, down = rnd(M["experts"], M["ff"], W), rnd(M["experts"], W, M["ff"])
+        for e in range(M["experts"]):
+            t[f"{p}mlp.e{e}.up"], t[f"{p}mlp.e{e}.down"] = up[e], down[e]
+        if M["shared"]:
+            t.update({p + "mlp.shared.up": rnd(M["shared"], W), p + "mlp.shared.down": rnd(W, M["shared"]), p + "mlp.shared.sg": rnd(1, W)})
+    model = importlib.import_module("llm-inference-engine_b200.models.vasolix").VasolixModel(config, t, **lb.limits)
+    touched, outputs = min(M["experts"], B * M["top"]), M["experts"] + (1 if M["shared"] else 0)
+    seen = lambda i: (i % chunk if chunk else i) + 1
+    att = W * (2 * H + Gk) * d + H * d * W
+    flops = 2.0 * Tq * 4 * (att + 2 * W * (M["top"] * M["ff"] + M["shared"]) + W * outputs) + 2.0 * 4 * 2 * H * d * float(sum(seen(i) for i in range(Tq)))
+    n_bytes = 2 * 4 * (att + 2 * W * (touched * M["ff"] + M["shared"]) + W * outputs) + 2 * V * W + 2.0 * 4 * 2 * B * Gk * d * seen(lb.ctx)
+    return model, flops, n_bytes
+
+
 def run_latent(args):
     """--mode latent: prefill and decode throughput of a Zefenex-shaped model (random weights, bf16) on the layer-list decoder at one of
     LATENT_SIZES and, in the same process, of the framework's closest other design at equal size: a Vasolix-shaped model of four chunked-
@@ -1288,15 +1323,13 @@ def run_latent(args):
     mod = importlib.import_module("llm-inference-engine_b200")
     mod.lib()
     sz = LATENT_SIZES[args.latent_size]
-    W, H, M, V = sz["width"], sz["heads"], sz["moe"], 32000
+    W, H, M = sz["width"], sz["heads"], sz["moe"]
     d, dr, r = sz["dim"], sz["rot"], sz["rank"]
     Tq, B, ctx = args.prefill_tokens, args.batch, args.ctx
     if ctx % sz["window"] == 0:
         ctx += sz["window"] // 2  # a context that ends exactly on a chunk edge would leave the chunked model's decoded token a single key to look at
     lb = LayerListBench(args, mod, ctx)
-    rnd, ones = lb.rnd, lb.ones
-    touched = min(M["experts"], B * M["top"])
-    window = sz["window"]
+    window, Gk = sz["window"], max(1, H // 4)
 
     # ---- the Zefenex-shaped model
     model, flops, n_bytes = zefenex_model(lb, sz)
@@ -1304,29 +1337,8 @@ def run_latent(args):
     del model
     torch.cuda.empty_cache()
 
-    # ---- the closest other design at equal size: four chunked-attention layers (values = keys, whole-projection norms), sigmoid-routed experts
-    att = {"type": "attention", "mixer": {"heads": H, "kv_heads": max(1, H // 4), "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": window}},
-           "mlp": {"kind": "moe", "expert": {"ff": M["ff"]}, "router": {"experts": M["experts"], "top": M["top"]}, "shared": {"ff": M["shared"]}}}
-    vconfig = {"architecture": "Vasolix", "layers": [att] * 4, "norm": {"eps": 1e-6}, "vocab": V, "width": W}
-    Gk = att["mixer"]["kv_heads"]
-    t = {"embed": rnd(V, W, std=1.0), "head": rnd(V, W), "final.norm": ones(W)}
-    for i in range(4):
-        p = f"l{i}."
-        t[p + "norm1"], t[p + "norm2"] = ones(W), ones(W)
-        t.update({p + "mix.q": rnd(H * d, W), p + "mix.k": rnd(Gk * d, W), p + "mix.g": rnd(H * d, W), p + "mix.o": rnd(W, H * d),
-                  p + "mix.q.norm": ones(H * d), p + "mix.k.norm": ones(Gk * d), p + "mix.sink": torch.zeros(H, dtype=torch.bfloat16)})
-        t[p + "mlp.router"] = rnd(M["experts"], W)
-        up, down = rnd(M["experts"], M["ff"], W), rnd(M["experts"], W, M["ff"])
-        for e in range(M["experts"]):
-            t[f"{p}mlp.e{e}.up"], t[f"{p}mlp.e{e}.down"] = up[e], down[e]
-        t.update({p + "mlp.shared.up": rnd(M["shared"], W), p + "mlp.shared.down": rnd(W, M["shared"]), p + "mlp.shared.sg": rnd(1, W)})
-    vas = importlib.import_module("llm-inference-engine_b200.models.vasolix")
-    vmodel = vas.VasolixModel(vconfig, t, **lb.limits)
-    v_att = W * (2 * H + Gk) * d + H * d * W
-    v_moe = 2 * W * (M["top"] * M["ff"] + M["shared"]) + W * (M["experts"] + 1)
-    chunk_pairs = float(sum(i % window + 1 for i in range(Tq)))
-    v_flops = 2.0 * Tq * 4 * (v_att + v_moe) + 2.0 * 4 * 2 * H * d * chunk_pairs
-    v_bytes = 2 * 4 * (v_att + 2 * W * (touched * M["ff"] + M["shared"]) + W * (M["experts"] + 1)) + 2 * V * W + 2.0 * 4 * 2 * B * Gk * d * (ctx % window + 1)
+    # ---- the closest other design at equal size
+    vmodel, v_flops, v_bytes = vasolix_model(lb, sz)
     closest = lb.measure(vmodel.engine, v_flops, v_bytes)
     print(json.dumps({
         "metric": "latent-attention model prefill / decode tokens/s", "value": latent["prefill"]["tokens_per_s"], "unit": "tokens/s (prefill)", "n_gpus": 1,
@@ -1424,6 +1436,89 @@ def run_zasapel(args):
         "e2e": "all numbers are taken through HybridDecoder.forward: host batch description in (one H2D copy per call), device logits out"}), flush=True)
 
 
+BEHIND_NORM_SIZES = {  # Pamulix-shaped layer lists (chunked attention / latent / chunked attention / latent, experts everywhere).  Widths, heads,
+    # ranks, windows (as chunks) and expert sizes follow LATENT_SIZES, so that the Zefenex- and Vasolix-shaped models of the same numbers (without
+    # identity experts and shared expert, which this design does not have) stand beside it.
+    "s": dict(LATENT_SIZES["s"], q_rank=384),
+    "m": dict(LATENT_SIZES["m"], q_rank=768),
+    "l": dict(LATENT_SIZES["l"], q_rank=1536),
+}
+
+
+def pamulix_model(lb, sz):
+    """The Pamulix-shaped model of the numbers `sz`, with the FLOPs of its prefill and the bytes of its decode step."""
+    import torch
+
+    rnd, ones, Tq, B, V = lb.rnd, lb.ones, lb.tokens, lb.batch, lb.vocab
+    W, H, M, rq, d, dr, dv, r, chunk = sz["width"], sz["heads"], sz["moe"], sz["q_rank"], sz["dim"], sz["rot"], sz["vdim"], sz["rank"], sz["chunk"]
+    G = max(1, H // 4)
+    moe = {"kind": "moe", "expert": {"ff": M["ff"]}, "router": {"experts": M["experts"], "top": M["top"]}}
+    att = {"type": "attention", "mlp": moe, "mixer": {"heads": H, "kv_heads": G, "dim": d, "vdim": dv, "scale": d ** -0.5, "mask": {"size": chunk}, "v_mix": True}}
+    rot = {"base": 10000.0, "dims": dr, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+    lat = {"type": "latent_attention", "mlp": moe, "mixer": {"heads": H, "dim": d, "rot_dim": dr, "vdim": dv, "kv_rank": r, "q_rank": rq, "scale": (d + dr) ** -0.5, "rot": rot}}
+    layers = [att, lat, att, lat]
+    config = {"architecture": "Pamulix", "width": W, "vocab": V, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "layers": layers}
+    t = {"embed": rnd(V, W, std=1.0), "head": rnd(V, W), "final.norm": ones(W)}
+    params = 0
+    for i, layer in enumerate(layers):
+        p = f"l{i}."
+        t.update({p + "norm1": ones(W), p + "norm2": ones(W), p + "mix.o": rnd(W, H * dv), p + "mlp.router": rnd(M["experts"], W),
+                  p + "mlp.router.b": torch.zeros(M["experts"], dtype=torch.bfloat16)})
+        params += W * H * dv
+        if layer["type"] == "attention":
+            t.update({p + "mix.q": rnd(H * d, W), p + "mix.k": rnd(G * d, W), p + "mix.v": rnd(G * dv, W), p + "mix.q.norm": ones(d), p + "mix.k.norm": ones(d),
+                      p + "mix.vmix": torch.tensor(0.5, dtype=torch.bfloat16)})
+            params += W * ((H + G) * d + G * dv)
+        else:
+            t.update({p + "mix.dq": rnd(rq, W), p + "mix.dq.norm": ones(rq), p + "mix.uq": rnd(H * (d + dr), rq), p + "mix.dkv": rnd(r + dr, W),
+                      p + "mix.dkv.norm": ones(r), p + "mix.uk": rnd(H * d, r, std=0.05), p + "mix.uv": rnd(H * dv, r, std=0.05)})
+            params += W * (rq + r + dr) + rq * H * (d + dr) + H * (d + dv) * r
+        gate, up, down = rnd(M["experts"], M["ff"], W), rnd(M["experts"], M["ff"], W), rnd(M["experts"], W, M["ff"])
+        for e in range(M["experts"]):
+            t[f"{p}mlp.e{e}.gate"], t[f"{p}mlp.e{e}.up"], t[f"{p}mlp.e{e}.down"] = gate[e], up[e], down[e]
+    model = importlib.import_module("llm-inference-engine_b200.models.pamulix").PamulixModel(config, t, **lb.limits)
+    touched = min(M["experts"], B * M["top"])
+    chunk_pairs = float(sum(i % chunk + 1 for i in range(Tq)))
+    flops = 2.0 * Tq * (params + 4 * (3 * W * M["top"] * M["ff"] + W * M["experts"])) + 2.0 * 2 * H * (d + dv) * chunk_pairs + \
+        2.0 * 2 * H * (2 * r + dr) * (Tq * (Tq + 1) / 2.0)
+    n_bytes = 2 * (params + 4 * (3 * W * touched * M["ff"] + W * M["experts"]) + V * W) + 2.0 * 2 * B * (G * (d + dv) * (lb.ctx % chunk + 1) + (r + dr) * (lb.ctx + 1))
+    return model, flops, n_bytes
+
+
+def run_pamulix(args):
+    """--mode pamulix: prefill and decode throughput of a Pamulix-shaped model (random weights, bf16) on the layer-list decoder at one of
+    BEHIND_NORM_SIZES and, in the same process, of the framework's two closest other designs at equal size: the Zefenex-shaped model (latent
+    attention, causal; softmax-routed gated experts) and the Vasolix-shaped one (chunked attention).  Prefill: one prompt of --prefill-tokens
+    tokens in one engine call.  Decode: --batch sequences with --ctx cached positions each, one token per sequence per step."""
+    import torch
+
+    mod = importlib.import_module("llm-inference-engine_b200")
+    mod.lib()
+    sz = BEHIND_NORM_SIZES[args.pamulix_size]
+    sz = dict(sz, chunk=sz["window"], moe=dict(sz["moe"], identity=0, shared=0))
+    W, H, M, rq, d, r, chunk = sz["width"], sz["heads"], sz["moe"], sz["q_rank"], sz["dim"], sz["rank"], sz["chunk"]
+    ctx = args.ctx + (chunk // 2 if args.ctx % chunk == 0 else 0)  # a context on a chunk edge would leave the decoded token a single key to look at
+    lb = LayerListBench(args, mod, ctx)
+    result = {}
+    models = {"pamulix": lambda: pamulix_model(lb, sz), "closest": lambda: zefenex_model(lb, dict(sz, window=0)), "closest_attention": lambda: vasolix_model(lb, sz)}
+    for name in ("pamulix",) if args.no_closest else models:
+        model, flops, n_bytes = models[name]()
+        result[name] = lb.measure(model.engine, flops, n_bytes)
+        del model
+        torch.cuda.empty_cache()
+    experts = f"{M['experts']} experts top {M['top']}"
+    print(json.dumps({
+        "metric": "norm-behind model prefill / decode tokens/s", "value": result["pamulix"]["prefill"]["tokens_per_s"], "unit": "tokens/s (prefill)", "n_gpus": 1,
+        "steps": args.steps, "warmup": max(args.warmup, 3), "higher_is_better": True, "dtype": "bf16", "data": "synthetic", "impl": "b200",
+        "config": {"model": f"Pamulix-shaped, size {args.pamulix_size}: width {W}, layers attention / latent / attention / latent ({H} heads, dim {d}; attention: {max(1, H // 4)} "
+                            f"kv heads, chunk {chunk}; latent: rotated {sz['rot']}, rank {r}, query rank {rq}, causal), 4 x {experts}",
+                   "closest": f"Zefenex-shaped: width {W}, 4 latent-attention layers ({H} heads, dim {d}+{sz['rot']}, rank {r}, causal), dense ff {sz['dense_ff']} + 3 x {experts}",
+                   "closest_attention": f"Vasolix-shaped: width {W}, 4 chunked-attention layers ({H} heads over {max(1, H // 4)} kv heads, dim {d}, chunk {chunk}), 4 x {experts}",
+                   "prefill_tokens": lb.tokens, "decode_batch": lb.batch, "decode_context": ctx, "cache_policy": "weights larger than L2 at sizes m and l; no explicit flush"},
+        **result,
+        "e2e": "all numbers are taken through HybridDecoder.forward: host batch description in (one H2D copy per call), device logits out"}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1441,8 +1536,9 @@ def main():
     ap.add_argument("--fedovik-size", default="m", choices=list(SHARED_NORM_SIZES), help="--mode fedovik: which Fedovik-shaped model")
     ap.add_argument("--silonex-size", default="m", choices=list(STREAM_SIZES), help="--mode silonex: which Silonex-shaped model")
     ap.add_argument("--zasapel-size", default="m", choices=list(SUM_NORM_SIZES), help="--mode zasapel: which Zasapel-shaped model")
-    ap.add_argument("--no-closest", action="store_true", help="--mode fedovik / silonex / zasapel: leave out the closest other model beside it")
-    ap.add_argument("--mode", default="decode", choices=["decode", "prefill", "generate", "serve", "hybrid", "latent", "fedovik", "silonex", "zasapel"],
+    ap.add_argument("--pamulix-size", default="m", choices=list(BEHIND_NORM_SIZES), help="--mode pamulix: which Pamulix-shaped model")
+    ap.add_argument("--no-closest", action="store_true", help="--mode fedovik / silonex / zasapel / pamulix: leave out the closest other model beside it")
+    ap.add_argument("--mode", default="decode", choices=["decode", "prefill", "generate", "serve", "hybrid", "latent", "fedovik", "silonex", "zasapel", "pamulix"],
                     help="decode (default, the BASELINE metric); prefill: one pass of --prefill-tokens tokens through all layers; generate: "
                          "the whole loop through b200_generate (prompt of --prefill-tokens tokens, --new-tokens sampled tokens, host in / host out)")
     ap.add_argument("--new-tokens", type=int, default=128)
@@ -1480,6 +1576,9 @@ def main():
         return
     if args.mode == "zasapel":
         run_zasapel(args)
+        return
+    if args.mode == "pamulix":
+        run_pamulix(args)
         return
     if args.mode == "fedovik":
         run_fedovik(args)

@@ -66,7 +66,33 @@ latent_prep_kernel(const T *__restrict__ proj, int ld, int q_col, int kv_col, T 
     };
     const int per = dim + rot_dim;
     constexpr int V = Elem<T>::kVec;
-    if (dim % V == 0 && rot_dim % V == 0 && ld % V == 0 && q_col % V == 0 &&
+    // neighbouring pairs lie inside one 16-byte piece: the piece at column c (from the rotated part's start) turns in registers
+    auto rotate_piece = [&](float *v, int c) {
+#pragma unroll
+        for (int i = 0; i < V; i += 2) {
+            if (c + i < rot_dims) {
+                const float a = v[i], b = v[i + 1], cv = cosv[(c + i) >> 1], sv = sinv[(c + i) >> 1];
+                v[i] = a * cv - b * sv, v[i + 1] = b * cv + a * sv;
+            }
+        }
+    };
+    if (rt.pairs && dim % V == 0 && rot_dim % V == 0 && ld % V == 0 && q_col % V == 0 &&
+        ((reinterpret_cast<size_t>(proj) | reinterpret_cast<size_t>(qn) | reinterpret_cast<size_t>(qr)) & 15) == 0) {
+        const int pieces = per / V;
+#pragma unroll 4
+        for (int idx = threadIdx.x; idx < heads * pieces; idx += blockDim.x) {
+            const int h = idx / pieces, c = (idx - h * pieces) * V;
+            const uint4 piece = ld_v4(row + q_col + (size_t)idx * V);
+            if (c < dim) {
+                st_v4(qn + ((size_t)h * t_pad + t) * dim + c, piece);
+            } else {
+                float v[V];
+                unpack16<T>(piece, v);
+                rotate_piece(v, c - dim);
+                st_v4(qr + ((size_t)t * heads + h) * rot_dim + (c - dim), pack16<T>(v));
+            }
+        }
+    } else if (dim % V == 0 && rot_dim % V == 0 && ld % V == 0 && q_col % V == 0 &&
         ((reinterpret_cast<size_t>(proj) | reinterpret_cast<size_t>(qn)) & 15) == 0) {  // the un-rotated part moves in 16-byte pieces
         const int pieces = dim / V;
         for (int idx = threadIdx.x; idx < heads * pieces; idx += blockDim.x) {
@@ -87,7 +113,31 @@ latent_prep_kernel(const T *__restrict__ proj, int ld, int q_col, int kv_col, T 
     }
     if (kv_col < 0) return;  // this layer reads another layer's rows
     const T *kv = (kv_proj ? kv_proj + (size_t)t * kv_ld : row) + kv_col;
+    const int rows_ld = kv_proj ? kv_ld : ld;
     float ss = 0.0f;
+    if (rt.pairs && kv_rank % V == 0 && rot_dim % V == 0 && rows_ld % V == 0 && kv_col % V == 0 && kv_rank + rot_dim <= (int)blockDim.x * V &&
+        ((reinterpret_cast<size_t>(kv_proj ? kv_proj : proj) | reinterpret_cast<size_t>(pool) | reinterpret_cast<size_t>(kv_norm)) & 15) == 0) {
+        const int c = threadIdx.x * V;  // one piece per thread, held between the sum and the scaling
+        float v[V];
+        if (c < kv_rank + rot_dim) unpack16<T>(ld_v4(kv + c), v);
+        if (c < kv_rank) {
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss);
+        }
+        const float inv = rsqrtf(block_sum(ss, red) / (float)kv_rank + eps);
+        const int page = block_table[(size_t)tok_seq[t] * mpps + pos / kPageL];
+        if (page < 0 || c >= kv_rank + rot_dim) return;  // no page held: nothing is written (the host refuses such a batch)
+        if (c < kv_rank) {
+            float w[V];
+            load_vec<V>(kv_norm + c, w);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] *= inv * w[e];
+        } else {
+            rotate_piece(v, c - kv_rank);
+        }
+        st_v4(pool + ((size_t)page * kPageL + (pos % kPageL)) * (kv_rank + rot_dim) + c, pack16<T>(v));
+        return;
+    }
     for (int c = threadIdx.x; c < kv_rank; c += blockDim.x) {
         const float v = Elem<T>::to_f(kv[c]);
         ss = fmaf(v, v, ss);

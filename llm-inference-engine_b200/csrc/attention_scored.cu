@@ -109,6 +109,63 @@ scored_prep_kernel(const T *__restrict__ proj, int ld, int col0, const float *__
     }
 }
 
+// The same step in 16-byte pieces, for layers without rotation, biases and value norm whose head rows are a power of two of pieces (at most a
+// warp): dim / V adjacent lanes share a head, its mean square is a shuffle sum among them.  One CTA per token.
+template <typename T>
+__global__ void __launch_bounds__(128)
+scored_prep_vec_kernel(const T *__restrict__ proj, int ld, int col0, T *__restrict__ q_out, T *__restrict__ k_pool, T *__restrict__ v_pool,
+                       const float *__restrict__ q_norm, const float *__restrict__ k_norm, float eps, const int *__restrict__ tok_seq,
+                       const int *__restrict__ tok_pos, const int *__restrict__ block_table, int mpps, int heads, int kv_heads, int dim, int vdim,
+                       T *__restrict__ v_keep, const T *__restrict__ v_mix, float lambda) {
+    constexpr int V = Elem<T>::kVec;
+    const int t = blockIdx.x, pos = tok_pos[t], per = dim / V, n_qk = (heads + kv_heads) * per, n_v = kv_heads * vdim / V;
+    const T *row = proj + (size_t)t * ld + col0;
+    const int page = block_table[(size_t)tok_seq[t] * mpps + pos / kPageS], off = pos % kPageS;
+#pragma unroll 3
+    for (int i0 = 0; i0 < n_qk; i0 += blockDim.x) {  // block-uniform trip count: the shuffles below take every lane
+        const int i = i0 + threadIdx.x, hh = i / per, c = (i - hh * per) * V;
+        const bool live = i < n_qk;
+        float v[V];
+        if (live) {
+            unpack16<T>(ld_v4(row + (size_t)i * V), v);
+        } else {
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] = 0.0f;
+        }
+        const float *nw = hh < heads ? q_norm : k_norm;
+        if (q_norm) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss);
+            for (int o = per >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            const float inv = rsqrtf(ss / (float)dim + eps);
+            if (live) {
+                float w[V];
+                load_vec<V>(nw + c, w);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[e] *= inv * w[e];
+            }
+        }
+        if (!live) continue;
+        if (hh < heads) st_v4(q_out + (size_t)t * heads * dim + (size_t)i * V, pack16<T>(v));
+        else if (page >= 0) st_v4(k_pool + (((size_t)page * kv_heads + (hh - heads)) * kPageS + off) * dim + c, pack16<T>(v));
+    }
+    for (int i = threadIdx.x; i < n_v; i += blockDim.x) {
+        const int g = i * V / vdim, c = i * V - g * vdim;
+        uint4 piece = ld_v4(row + (size_t)n_qk * V + (size_t)i * V);
+        if (v_keep) st_v4(v_keep + ((size_t)t * n_v + i) * V, piece);
+        if (v_mix) {
+            float v[V], f[V];
+            unpack16<T>(piece, v);
+            unpack16<T>(ld_v4(v_mix + ((size_t)t * n_v + i) * V), f);
+#pragma unroll
+            for (int e = 0; e < V; ++e) v[e] = (1.0f - lambda) * v[e] + lambda * f[e];
+            piece = pack16<T>(v);
+        }
+        if (page >= 0) st_v4(v_pool + (((size_t)page * kv_heads + g) * kPageS + off) * vdim + c, piece);
+    }
+}
+
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 // for weights that are rounded to 16 bits right away: hardware exponential and reciprocal (relative error ~1e-6)
 __device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
@@ -561,6 +618,15 @@ int launch_scored_prep(int dtype, const void *proj, int ld, int col0, const floa
                        ScoredPrepOptions opt, ValueShare share) {
     if (tokens == 0) return B200_OK;
     B200_DISPATCH_DTYPE(dtype, {
+        constexpr int V = Elem<T>::kVec;
+        const int per = dim / V;
+        if (rot_dims == 0 && !b_in && !opt.v_norm && dim % V == 0 && per <= 32 && (per & (per - 1)) == 0 && vdim % V == 0 && ld % V == 0 && col0 % V == 0 &&
+            (q_norm == nullptr) == (k_norm == nullptr) && all_aligned16({proj, q_out, k_pool, v_pool, q_norm, k_norm, share.v_keep, share.v_mix})) {
+            scored_prep_vec_kernel<T><<<tokens, 128, 0, st>>>((const T *)proj, ld, col0, (T *)q_out, (T *)k_pool, (T *)v_pool, q_norm, k_norm, eps,
+                                                              tok_seq, tok_pos, block_table, mpps, heads, kv_heads, dim, vdim, (T *)share.v_keep,
+                                                              (const T *)share.v_mix, share.lambda);
+            return cuda_status("scored_prep (vector) launch");
+        }
         scored_prep_kernel<T><<<tokens, 256, (size_t)std::max(rot_dims, 2) * sizeof(float), st>>>(
             (const T *)proj, ld, col0, b_in, (T *)q_out, (T *)k_pool, (T *)v_pool, q_norm, k_norm, eps, tok_seq, tok_pos, block_table, mpps, heads,
             kv_heads, dim, vdim, rot_dims, rot_base, opt, (T *)share.v_keep, (const T *)share.v_mix, share.lambda);

@@ -9,6 +9,7 @@
 #include <stdio.h>
 #include <stdarg.h>
 #include <string.h>
+#include <initializer_list>
 
 #include "../../include/b200llm.h"
 
@@ -42,6 +43,11 @@ struct NvtxRange {
 #endif
 
 inline bool aligned16(const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
+inline bool all_aligned16(std::initializer_list<const void *> ps) {
+    for (const void *p : ps)
+        if (!aligned16(p)) return false;
+    return true;
+}
 inline cudaStream_t as_stream(b200_stream_t s) { return reinterpret_cast<cudaStream_t>(s); }
 
 // Library workspace (device memory, caller- or library-owned): [tickets | scratch].
@@ -342,6 +348,7 @@ __device__ __forceinline__ void tp_reduce_vec(const TpExchange &t, unsigned int 
 
 // N (1 or 4) consecutive elements of T <-> fp32; N == 4: one 16-byte (fp32) or 8-byte (16-bit) access, the address aligned to it
 template <typename T, int N> __device__ __forceinline__ void load_n(const T *__restrict__ p, float *v) {
+    static_assert(N == 1 || N == 4, "load_n takes 1 or 4 elements");
     if constexpr (N == 1) {
         v[0] = Elem<T>::to_f(p[0]);
     } else if constexpr (sizeof(T) == 4) {
@@ -355,6 +362,7 @@ template <typename T, int N> __device__ __forceinline__ void load_n(const T *__r
     }
 }
 template <typename T, int N> __device__ __forceinline__ void store_n(T *__restrict__ p, const float *v) {
+    static_assert(N == 1 || N == 4, "store_n takes 1 or 4 elements");
     if constexpr (N == 1) {
         p[0] = Elem<T>::from_f(v[0]);
     } else if constexpr (sizeof(T) == 4) {
@@ -365,6 +373,14 @@ template <typename T, int N> __device__ __forceinline__ void store_n(T *__restri
 #pragma unroll
         for (int i = 0; i < 4; ++i) e[i] = Elem<T>::from_f(v[i]);
         *reinterpret_cast<uint2 *>(p) = raw;
+    }
+}
+// N (a multiple of 4) consecutive floats, the address 16-byte aligned
+template <int N> __device__ __forceinline__ void load_vec(const float *__restrict__ p, float *v) {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+        const float4 a = *reinterpret_cast<const float4 *>(p + i);
+        v[i] = a.x, v[i + 1] = a.y, v[i + 2] = a.z, v[i + 3] = a.w;
     }
 }
 // ------------------------------------------------------------------ activations (b200_act_t)

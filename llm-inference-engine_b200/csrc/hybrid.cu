@@ -159,14 +159,6 @@ template <int N> __device__ __forceinline__ void dyt_apply_vec(const float *__re
         v[i + 2] = fmaf(dyt_tanh(alpha * v[i + 2]), w.z, b.z), v[i + 3] = fmaf(dyt_tanh(alpha * v[i + 3]), w.w, b.w);
     }
 }
-template <int N> __device__ __forceinline__ void load_vec(const float *__restrict__ p, float *v) {
-#pragma unroll
-    for (int i = 0; i < N; i += 4) {
-        const float4 a = *reinterpret_cast<const float4 *>(p + i);
-        v[i] = a.x, v[i + 1] = a.y, v[i + 2] = a.z, v[i + 3] = a.w;
-    }
-}
-
 // The general form of the kernel above, for either norm kind and either place of the routing weights:
 //   y[t, :]  = y_dense[t, :] + y_bias                                                  (a dense sublayer), or
 //            = sum_k w(t, k) * (pair_row[t, k] >= 0 ? y_rows[pair_row[t, k], :] : h_in[t, :]) + shared_gate[t] * y_shared[t, :]

@@ -270,12 +270,6 @@ conv_input_kernel(const float *__restrict__ x, T *__restrict__ h, int width, int
     }
 }
 
-static bool all_aligned16(std::initializer_list<const void *> ps) {
-    for (const void *p : ps)
-        if ((reinterpret_cast<size_t>(p) & 15) != 0) return false;
-    return true;
-}
-
 int launch_sum_norm(int dtype, float *x, const void *y_dense, const void *y_rows, const int *pair_row, int top, const void *y_shared,
                     const float *shared_gate, float alpha, const float *g, float eps, int width, float *trace, void *h_out, RingConv own, RingConv next,
                     int one_token, PortionMap pm, int tokens, cudaStream_t st) {
