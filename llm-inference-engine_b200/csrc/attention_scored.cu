@@ -329,7 +329,8 @@ scored_attn_kernel(const T *__restrict__ q, const T *__restrict__ k_pool, const 
 // of 16 rows each.  A key tile is one page (64 positions): K and V arrive by cp.async into a two-stage ring, S = Q K^T and O += P V run on
 // mma.sync.m16n8k16 with fp32 accumulators.  SOFTMAX: the online form in fp32 (base 2); the distance penalty of a head is a table over the
 // distance in shared memory.  SIGMOID: P = sigmoid(score + head_bias) goes to the second product as it is: no running state at all.
-// The mask is evaluated per element; the tiles walked are those from the window start of the tile's first query to its last query.
+// A linear distance bias is one more fused multiply-add per score; a sink is the initial running state.  The mask (window, blocks) is evaluated
+// per element; the tiles walked are those from the first key the tile's first query sees to its last query.
 // tiles: int4 per tile {sequence, first packed row, rows (1..64), position of the first row}.
 constexpr int kTileQS = 64;
 

@@ -7,7 +7,8 @@
 //            the worst-case number of tiles and the surplus CTAs leave at once.
 //   gather:  row <- T(weight * x[token])  -- the weight multiplies the expert's input, which matters for a non-linear expert;
 //   grouped GEMM (x2): up with the activation in the epilogue, then down.
-// A second router form (softmax): scores = softmax(router logits) over all router outputs; the choice is made on score + a per-expert bias,
+// A second router form (softmax): scores = softmax(router logits + an optional bias) over all router outputs; the choice is made on score + a
+// per-expert choice bias (without one: on the logit),
 // the weights are the chosen experts' scores divided by their sum and multiply the expert's OUTPUT; router outputs past the real experts
 // are identity experts (they return their input and own no rows of the grouped GEMM); experts may be gated: act(gate rows) * up rows.
 // The sum over a token's experts, the shared expert and the post-norm are one kernel of the engine (hybrid.cu).

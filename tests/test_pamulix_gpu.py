@@ -448,11 +448,11 @@ def test_rotated_part_alone_finds_its_distance(back, decode, dtype):
 def test_tensor_core_paths_against_the_oracle_and_against_single_tokens(dtype):
     """Sizes every tensor-core path takes: tiles of prompt tokens in blocks that end inside a tile and inside a page, one-token tiles over 20
     heads, a rank of 256, head products and experts on 128-row tiles (a prompt of 300 tokens), 16-byte pieces everywhere."""
-    layers = [ref.attention(heads=4, kv_heads=2, dim=64, vdim=32, chunk=90, mlp=ref.moe(experts=4, top=4, ff=64)),
-              ref.latent(heads=6, dim=64, rot_dim=16, vdim=48, kv_rank=80, q_rank=64, mlp=ref.moe(experts=4, top=4, ff=64)),
-              ref.attention(heads=8, kv_heads=2, dim=128, vdim=32, chunk=37),
+    layers = [ref.attention(heads=6, kv_heads=3, dim=64, vdim=32, chunk=90, mlp=ref.moe(experts=4, top=4, ff=64)),
+              ref.latent(heads=5, dim=64, rot_dim=16, vdim=48, kv_rank=80, q_rank=64, mlp=ref.moe(experts=4, top=4, ff=64)),
+              ref.attention(heads=9, kv_heads=3, dim=128, vdim=32, chunk=37),
               ref.latent(heads=20, dim=64, rot_dim=32, vdim=64, kv_rank=80, q_rank=96),
-              ref.attention(heads=2, kv_heads=2, dim=32, vdim=32, chunk=350),
+              ref.attention(heads=3, kv_heads=3, dim=32, vdim=32, chunk=350),
               ref.latent(heads=2, dim=64, rot_dim=16, vdim=24, kv_rank=256, q_rank=64, scale=0.1)]
     config = ref.make_config(layers, width=64)
     W, packed = ref.make_weights(config, seed=41)
